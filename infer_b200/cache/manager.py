@@ -6,11 +6,12 @@ launches nothing (the reference keeps the same split, src/block_pool.h:14-15).  
 are made by ``make_storage`` and handed to the parts as views.
 
 Groups.  Every cache entry of the run order states a need (``PagedKVNeed`` / ``StateNeed`` / none).
-Paged entries with the same (kv heads, key and value size, window) form a *group*: the group has one page
+Paged entries with the same (kv heads, key and value size, window, chunk) form a *group*: the group has one page
 pool and one block table per request, and a page id addresses the same page in every entry of the
 group (the reference has one implicit group: one block id spans all layers,
 kernels/batch_gpu.cu:75,114-118).  Groups with a window give pages back as soon as every later
-query is past them; their block tables then hold -1 at that place.  A need with ``keep_first`` keeps the pages
+query is past them; their block tables then hold -1 at that place.  Groups with chunks (a query reads keys of its own
+chunk of positions only) give back the pages of the chunks that have passed.  A need with ``keep_first`` keeps the pages
 that hold the positions below it: every later query still reads those.
 
 An entry may also state a ``CompositeNeed``: several needs by name (pages AND a fixed-size state for one mixer;
@@ -132,7 +133,7 @@ class CacheManager:
             """key: the cache index, or (cache index, name, ...) for a leaf of a composite need."""
             if isinstance(need, PagedKVNeed):
                 gkey = (need.num_kv_heads, need.head_dim, need.value_dim, need.window, need.values_in_keys,
-                        need.keep_first if need.window is not None else 0)
+                        need.keep_first if need.window is not None else 0, need.chunk)
                 g = by_key.get(gkey)
                 if g is None:
                     g = CacheGroup(len(self.groups), need, [], PagePool(n_pages), page_size)
@@ -215,9 +216,10 @@ class CacheManager:
 
     def _first_needed_page(self, g: CacheGroup, length: int) -> int:
         """Index of the first page that a query at position >= length can still read."""
-        if g.window is None:
-            return 0
-        return max(0, length - g.window + 1) // self.page_size
+        first = 0 if g.window is None else max(0, length - g.window + 1)
+        if g.need.chunk is not None:
+            first = max(first, length // g.need.chunk * g.need.chunk)
+        return first // self.page_size
 
     def pages_needed(self, rid, n_new: int) -> List[int]:
         """Per group: pages that reserve(rid, n_new) would take from the pool."""

@@ -32,7 +32,7 @@ class PartSpec:
 
 
 # The families a part can belong to; each has its own registry of kinds (``parts.base``).
-FAMILIES = ("mixer", "feed_forward", "norm", "position", "block", "embedding", "head", "gate")
+FAMILIES = ("mixer", "feed_forward", "norm", "position", "block", "embedding", "head", "gate", "connection", "stream")
 
 
 @dataclass(frozen=True)
@@ -92,12 +92,15 @@ class ModelSpec:
     head: PartSpec                   # family "head": normalised rows -> float32 logits; may be tied to the embedding
     eos_token_id: Optional[int] = None
     optional_tensors: Sequence[str] = ()   # names a checkpoint may hold although no part reads them
+    stream: Optional[PartSpec] = None      # family "stream": a residual stream that is more than one row per token (None: it is one)
 
     def part_specs(self) -> Iterator[Tuple[str, PartSpec]]:
         """Every (family, PartSpec) of the model: embedding, head, final norm, then the layers' parts in order."""
         yield "embedding", self.embedding
         yield "head", self.head
         yield "norm", self.final_norm
+        if self.stream is not None:
+            yield "stream", self.stream
         for layer in self.layers:
             yield from layer.parts.values()
 

@@ -33,6 +33,8 @@ MODULES: Dict[str, str] = {
     "mix": "mix_ops.cu",         # norms on sublayer results, decayed and delta-rule recurrences, routers, row norms of q and k
     "latent": "latent_ops.cu",   # attention through low-rank latents, layer norm, sigmoid router, capped logits
     "post": "post_ops.cu",       # norms after the residual sum, per-head query/key norms, mixtures with the token before
+    "stream": "stream_ops.cu",   # several residual streams, norms over groups of channels, sinusoidal positions
+    "talk": "talk_ops.cu",       # attention whose heads exchange their scores before the softmax
     "latent_pf": "latent_prefill.cu",   # the same attention for prompt portions: per-head keys and values, tensor cores
     "gemvb": "gemv_bulk.cu",
     "gemm": "gemm_tcgen05.cu",

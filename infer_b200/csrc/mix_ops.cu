@@ -183,13 +183,15 @@ __global__ void glu_act_vec_kernel(const bf16* __restrict__ rows, int64_t ld, in
 }
 
 // ------------------------------------------------------------------------------------------------
-// Router: scores = softmax(logits) over all experts; experts form n_groups groups of neighbours, a group's score is
-// its largest; only experts of the `keep` best groups can be chosen; the `top` largest of those are chosen (ties:
-// the lower index); their weights are their scores divided by (their sum + sum_eps). One warp per token.
+// Router: scores = softmax(logits) over all experts, or the logits' sigmoids; experts form n_groups groups of neighbours,
+// a group's score is its largest, or the sum of its two largest (of its one, if it has one); only experts of the `keep`
+// best groups can be chosen; the `top` largest of those are chosen (ties: the lower index); their weights are their
+// scores divided by (their sum + sum_eps), or as they are, times `mult`. One warp per token.
 // weights [tokens, experts]: a chosen expert's weight, zero elsewhere. chosen [tokens, top] (optional): the indices.
 __global__ void __launch_bounds__(128)
 route_kernel(const float* __restrict__ logits, int64_t n_tokens, int n_experts, int top, int n_groups, int keep,
-             float sum_eps, float* __restrict__ weights, int* __restrict__ chosen) {
+             float sum_eps, int sigmoid, int group_best, int renormalise, float mult, float* __restrict__ weights,
+             int* __restrict__ chosen) {
     ib::pdl_wait();
     extern __shared__ float sm[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -198,24 +200,32 @@ route_kernel(const float* __restrict__ logits, int64_t n_tokens, int n_experts, 
     float* s = sm + warp * (n_experts + n_groups);          // scores; a chosen expert's score becomes -(1 + score)
     float* gs = s + n_experts;                               // group scores; -1: a kept group, -2: not kept
     const float* z = logits + t * n_experts;
-    float mx = -INFINITY;
-    for (int e = lane; e < n_experts; e += 32) mx = fmaxf(mx, z[e]);
-    mx = ib::warp_max(mx);
-    float sum = 0.0f;
-    for (int e = lane; e < n_experts; e += 32) {
-        const float v = expf(z[e] - mx);
-        s[e] = v;
-        sum += v;
+    if (sigmoid) {
+        for (int e = lane; e < n_experts; e += 32) s[e] = sigmoid_(z[e]);
+    } else {
+        float mx = -INFINITY;
+        for (int e = lane; e < n_experts; e += 32) mx = fmaxf(mx, z[e]);
+        mx = ib::warp_max(mx);
+        float sum = 0.0f;
+        for (int e = lane; e < n_experts; e += 32) {
+            const float v = expf(z[e] - mx);
+            s[e] = v;
+            sum += v;
+        }
+        sum = ib::warp_sum(sum);
+        __syncwarp();
+        for (int e = lane; e < n_experts; e += 32) s[e] = s[e] / sum;
     }
-    sum = ib::warp_sum(sum);
-    __syncwarp();
-    for (int e = lane; e < n_experts; e += 32) s[e] = s[e] / sum;
     __syncwarp();
     const int per = n_experts / n_groups;
     for (int g = lane; g < n_groups; g += 32) {
-        float m = -1.0f;
-        for (int j = 0; j < per; j++) m = fmaxf(m, s[g * per + j]);
-        gs[g] = m;
+        float m = -1.0f, m2 = -1.0f;                         // the two largest
+        for (int j = 0; j < per; j++) {
+            const float v = s[g * per + j];
+            if (v > m) { m2 = m; m = v; }
+            else m2 = fmaxf(m2, v);
+        }
+        gs[g] = (group_best == 2 && per > 1) ? m + m2 : m;
     }
     __syncwarp();
     for (int r = 0; r < keep; r++) {
@@ -254,7 +264,7 @@ route_kernel(const float* __restrict__ logits, int64_t n_tokens, int n_experts, 
         }
         __syncwarp();
     }
-    const float inv = 1.0f / (total + sum_eps);
+    const float inv = renormalise ? mult / (total + sum_eps) : mult;
     for (int e = lane; e < n_experts; e += 32) weights[t * n_experts + e] = s[e] < 0.0f ? (-1.0f - s[e]) * inv : 0.0f;
 }
 
@@ -636,7 +646,11 @@ __device__ __forceinline__ float filtered(const float* __restrict__ rows, int64_
 // sqrt(sum(x^2) + unit_eps), q also times q_scale; per head h: beta = sigmoid(raw[b_col + h]),
 // g = exp(-exp(a_log[h]) * softplus(raw[a_col + h] + dt_bias[h])).
 // prep rows (float, ldp): [q | k | v | g (H) | beta (H) | k.q (G)].
-// One warp per (token, unit): G units of a (q, k) head pair, H units of a v head, one unit for the heads' scalars.
+// With `z` (rows of H x d logits from column z_col, leading dimension ldz) the decay is a number per head and key
+// channel, g = exp(-exp(a_log[h]) * softplus(z[h d + i] + dt_bias[h d + i])), and the prep rows are
+// [q | k | v | up to 4 | g (H x d) | beta (H) | k.q (G)].
+// One warp per (token, unit): G units of a (q, k) head pair, H units of a v head, one unit for the heads' scalars, and
+// with `z` H units of a head's decays.
 constexpr int PREP_PER_LANE = 8;         // heads of up to 32 * PREP_PER_LANE channels
 
 // The newest input of channel c joins its request's tail, the oldest leaves (steps of one token per request: the lane
@@ -651,10 +665,11 @@ delta_prepare_kernel(const float* __restrict__ rows, int64_t ld, int col0, int a
                      const float* __restrict__ filt_w, int taps, float* tails, int inline_tail,
                      const float* __restrict__ a_log, const float* __restrict__ dt_bias, float unit_eps, float q_scale,
                      const int* __restrict__ token_seg, const int* __restrict__ seg_start, const int* __restrict__ seg_slot,
-                     float* __restrict__ prep, int64_t ldp, int64_t n_tokens, int n_heads, int n_qk, int d, int dv) {
+                     float* __restrict__ prep, int64_t ldp, int64_t n_tokens, int n_heads, int n_qk, int d, int dv,
+                     const float* __restrict__ z, int64_t ldz, int z_col) {
     ib::pdl_wait();
     const int lane = threadIdx.x & 31;
-    const int units = n_qk + n_heads + 1;
+    const int units = n_qk + n_heads + 1 + (z ? n_heads : 0);
     const int64_t wi = int64_t(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (wi >= n_tokens * units) return;
     const int64_t t = wi / units;
@@ -665,8 +680,16 @@ delta_prepare_kernel(const float* __restrict__ rows, int64_t ld, int col0, int a
     float* tail = taps > 1 ? tails + (int64_t(seg_slot[s]) * (taps - 1)) * channels : nullptr;
     const bool move = inline_tail && taps > 1;
     float* out = prep + t * ldp;
-    const int g_off = 2 * n_qk * d + n_heads * dv;
-    if (u < n_qk) {
+    const int g_off = z ? (2 * n_qk * d + n_heads * dv + 3) / 4 * 4 : 2 * n_qk * d + n_heads * dv;
+    const int beta_off = g_off + (z ? n_heads * d : n_heads);
+    if (u > n_qk + n_heads) {
+        const int h = u - n_qk - n_heads - 1;
+        const float rate = expf(a_log[h]);
+        for (int j = lane; j < d; j += 32) {
+            const int c = h * d + j;
+            out[g_off + c] = expf(-rate * softplus_(z[t * ldz + z_col + c] + dt_bias[c]));
+        }
+    } else if (u < n_qk) {
         float qv[PREP_PER_LANE], kv[PREP_PER_LANE];
         float sq = 0.0f, sk = 0.0f, dot = 0.0f;
 #pragma unroll
@@ -698,7 +721,7 @@ delta_prepare_kernel(const float* __restrict__ rows, int64_t ld, int col0, int a
                 out[n_qk * d + u * d + j] = kv[r] * fk;
             }
         }
-        if (lane == 0) out[g_off + 2 * n_heads + u] = dot * fq * fk;
+        if (lane == 0) out[beta_off + n_heads + u] = dot * fq * fk;
     } else if (u < n_qk + n_heads) {
         const int h = u - n_qk;
         for (int j = lane; j < dv; j += 32) {
@@ -708,9 +731,8 @@ delta_prepare_kernel(const float* __restrict__ rows, int64_t ld, int col0, int a
         }
     } else {
         for (int h = lane; h < n_heads; h += 32) {
-            const float a = rows[t * ld + a_col + h], b = rows[t * ld + b_col + h];
-            out[g_off + h] = expf(-expf(a_log[h]) * softplus_(a + dt_bias[h]));
-            out[g_off + n_heads + h] = sigmoid_(b);
+            if (!z) out[g_off + h] = expf(-expf(a_log[h]) * softplus_(rows[t * ld + a_col + h] + dt_bias[h]));
+            out[beta_off + h] = sigmoid_(rows[t * ld + b_col + h]);
         }
     }
 }
@@ -742,9 +764,13 @@ __global__ void tail_update_kernel(const float* __restrict__ rows, int64_t ld, i
 //   MODE 2 (a constant decay per head):  S <- g S + k_t v_t^T;                       o_t = S^T q_t
 //   MODE 3 (a decay per key channel, a bonus for the current token):
 //                                       o_t = (S + diag(u) k_t v_t^T)^T q_t;  then  S <- diag(a_t) S + k_t v_t^T
+//   MODE 4 (delta rule, a decay per key channel):
+//                                       S <- diag(a_t) S;  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t
 // MODE 1 is computed from the old state in one sweep: r = S^T k, p = S^T q, u = beta (v - g r), o = g p + u (k.q),
 // S <- g S + k u^T, with k.q given per token (aux rows). MODE 2 reads g at aux_col + h of the token's aux row (a
 // leading dimension of 0: one row for every token). MODE 3 reads its decays as MODE 0 and u [heads, d] from `bonus`.
+// MODE 4 reads its decays as MODE 0, beta at scal_col + h and k.q at scal_col + H + h / heads_per_qk of the same aux
+// rows, and works in one sweep as MODE 1: S <- diag(a) S with r = S^T k and p = S^T q, then S <- S + k u^T, o = p + u (k.q).
 // A column of S belongs to LK = 8 neighbouring lanes, lane j of them keeping rows j R .. j R + R - 1 in registers
 // (R >= d / 8, rows beyond d are zero and stay zero); a warp has 4 columns, a CTA `cb` columns of one (segment, head).
 // Column sums are added within a lane in four chains and across the 8 lanes by shuffles, in an order that depends on
@@ -764,21 +790,20 @@ __device__ __forceinline__ void copy_async4(float* smem_dst, const float* gmem_s
 // One token's operands of a thread: its R rows of q, k (and of the decays), the value of its column, the scalars.
 template <int R, int MODE>
 struct ScanOperands {
-    float4 q[R / 4], k[R / 4], a[(MODE == 0 || MODE == 3) ? R / 4 : 1];
+    float4 q[R / 4], k[R / 4], a[(MODE == 0 || MODE == 3 || MODE == 4) ? R / 4 : 1];
     float v, g, beta, kq;
-    __device__ __forceinline__ void load(const float* qs, const float* ks, const float* as, const float* vs, int c, int dpp, int off,
-                                         int cb, int col_l) {
+    __device__ __forceinline__ void load(const float* qs, const float* ks, const float* as, const float* ss, const float* vs, int c,
+                                         int dpp, int off, int cb, int col_l) {
         const float4* q4 = reinterpret_cast<const float4*>(qs + c * dpp + off);
         const float4* k4 = reinterpret_cast<const float4*>(ks + c * dpp + off);
 #pragma unroll
         for (int i = 0; i < R / 4; i++) { q[i] = q4[i]; k[i] = k4[i]; }
-        if (MODE == 0 || MODE == 3) {
+        if (MODE == 0 || MODE == 3 || MODE == 4) {
             const float4* a4 = reinterpret_cast<const float4*>(as + c * dpp + off);
 #pragma unroll
             for (int i = 0; i < R / 4; i++) a[i] = a4[i];
-        } else {
-            g = as[c * 4 + 0]; beta = as[c * 4 + 1]; kq = as[c * 4 + 2];
         }
+        if (MODE == 1 || MODE == 2 || MODE == 4) { g = ss[c * 4 + 0]; beta = ss[c * 4 + 1]; kq = ss[c * 4 + 2]; }
         v = vs[c * cb + col_l];
     }
 };
@@ -849,6 +874,42 @@ __device__ __forceinline__ float scan_token(float (&S)[R], const ScanOperands<R,
         p += __shfl_xor_sync(0xffffffffu, p, 4);
         return p;
     }
+    if (MODE == 4) {
+        float r0 = 0.0f, r1 = 0.0f, p0 = 0.0f, p1 = 0.0f;
+#pragma unroll
+        for (int i4 = 0; i4 < R / 4; i4++) {
+            const float4 a = x.a[i4], k = x.k[i4], q = x.q[i4];
+            S[4 * i4 + 0] *= a.x;
+            S[4 * i4 + 1] *= a.y;
+            S[4 * i4 + 2] *= a.z;
+            S[4 * i4 + 3] *= a.w;
+            r0 = fmaf(S[4 * i4 + 0], k.x, r0);
+            r1 = fmaf(S[4 * i4 + 1], k.y, r1);
+            r0 = fmaf(S[4 * i4 + 2], k.z, r0);
+            r1 = fmaf(S[4 * i4 + 3], k.w, r1);
+            p0 = fmaf(S[4 * i4 + 0], q.x, p0);
+            p1 = fmaf(S[4 * i4 + 1], q.y, p1);
+            p0 = fmaf(S[4 * i4 + 2], q.z, p0);
+            p1 = fmaf(S[4 * i4 + 3], q.w, p1);
+        }
+        float r = r0 + r1, p = p0 + p1;
+        r += __shfl_xor_sync(0xffffffffu, r, 1);
+        p += __shfl_xor_sync(0xffffffffu, p, 1);
+        r += __shfl_xor_sync(0xffffffffu, r, 2);
+        p += __shfl_xor_sync(0xffffffffu, p, 2);
+        r += __shfl_xor_sync(0xffffffffu, r, 4);
+        p += __shfl_xor_sync(0xffffffffu, p, 4);
+        const float u = x.beta * (v - r);
+#pragma unroll
+        for (int i4 = 0; i4 < R / 4; i4++) {
+            const float4 k = x.k[i4];
+            S[4 * i4 + 0] = fmaf(k.x, u, S[4 * i4 + 0]);
+            S[4 * i4 + 1] = fmaf(k.y, u, S[4 * i4 + 1]);
+            S[4 * i4 + 2] = fmaf(k.z, u, S[4 * i4 + 2]);
+            S[4 * i4 + 3] = fmaf(k.w, u, S[4 * i4 + 3]);
+        }
+        return fmaf(u, x.kq, p);
+    }
     const float g = x.g;
     float r0 = 0.0f, r1 = 0.0f, p0 = 0.0f, p1 = 0.0f;
 #pragma unroll
@@ -893,18 +954,20 @@ state_scan_kernel(const float* __restrict__ rows, int64_t ld, int q_col, int k_c
                   const float* __restrict__ aux, int64_t lda, int aux_col, float* __restrict__ state,
                   const int* __restrict__ seg_start, const int* __restrict__ seg_slot, float* __restrict__ raw_out,
                   int n_heads, int heads_per_qk, int d, int dv, int cb, int chunk, int write_state, int pipelined,
-                  const float* __restrict__ bonus, int act) {
+                  const float* __restrict__ bonus, int act, int scal_col) {
     extern __shared__ __align__(16) float sm[];
     constexpr int RP = R + 4, DPP = LK * RP;
-    constexpr bool ROWS = MODE == 0 || MODE == 3;      // the decays are rows like q and k
-    constexpr int N_SCAL = MODE == 1 ? 3 : 1;          // scalars per token otherwise
+    constexpr bool ROWS = MODE == 0 || MODE == 3 || MODE == 4;      // the decays are rows like q and k
+    constexpr bool SCAL = MODE == 1 || MODE == 2 || MODE == 4;      // scalars per token: [g, beta, k.q] in places 0..2
+    constexpr int SCAL0 = MODE == 4 ? 1 : 0, SCAL1 = MODE == 2 ? 1 : 3;     // the places that this mode has
     const int n_buf = pipelined ? 2 : 1;
-    const int a_tok = ROWS ? DPP : 4;
+    const int a_tok = ROWS ? DPP : 0, s_tok = SCAL ? 4 : 0;
     float* qs = sm;                          // [n_buf][chunk][DPP]
     float* ks = qs + n_buf * chunk * DPP;
-    float* as = ks + n_buf * chunk * DPP;    // MODE 0: [n_buf][chunk][DPP] decays; MODE 1: [n_buf][chunk][4] g, beta, k.q
-    float* vs = as + n_buf * chunk * a_tok;  // [n_buf][chunk][cb]
-    const int total = n_buf * chunk * (2 * DPP + a_tok + cb);
+    float* as = ks + n_buf * chunk * DPP;    // ROWS: [n_buf][chunk][DPP] decays
+    float* ss = as + n_buf * chunk * a_tok;  // SCAL: [n_buf][chunk][4] g, beta, k.q
+    float* vs = ss + n_buf * chunk * s_tok;  // [n_buf][chunk][cb]
+    const int total = n_buf * chunk * (2 * DPP + a_tok + s_tok + cb);
     const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
     const int hq = h / heads_per_qk;
     const int lk = tid & (LK - 1), col_l = tid >> 3;
@@ -926,6 +989,10 @@ state_scan_kernel(const float* __restrict__ rows, int64_t ld, int q_col, int k_c
     }
     __syncthreads();
 
+    auto scalar_at = [&](int e) -> int {     // column of scalar e in a token's aux row
+        if (MODE == 4) return scal_col + (e == 1 ? h : n_heads + hq);
+        return aux_col + (e == 0 ? h : (e == 1 ? n_heads + h : 2 * n_heads + hq));
+    };
     auto request = [&](int c0, int b) {      // asynchronous copies of the chunk that starts at token c0 into buffer b
         const int n = min(chunk, len - c0);
         const int d4 = d / 4, cb4 = cb / 4;
@@ -937,11 +1004,11 @@ state_scan_kernel(const float* __restrict__ rows, int64_t ld, int q_col, int k_c
             copy_async16(ks + dst, row + k_col + hq * d + j);
             if (ROWS) copy_async16(as + dst, aux + (t0 + c0 + c) * lda + aux_col + h * d + j);
         }
-        if (!ROWS) {
+        if (SCAL) {
+            constexpr int N_SCAL = SCAL1 - SCAL0;
             for (int idx = tid; idx < n * N_SCAL; idx += blockDim.x) {
-                const int c = idx / N_SCAL, e = idx - c * N_SCAL;
-                const float* ar = aux + (t0 + c0 + c) * lda + aux_col;
-                copy_async4(as + (b * chunk + c) * 4 + e, ar + (e == 0 ? h : (e == 1 ? n_heads + h : 2 * n_heads + hq)));
+                const int c = idx / N_SCAL, e = idx - c * N_SCAL + SCAL0;
+                copy_async4(ss + (b * chunk + c) * 4 + e, aux + (t0 + c0 + c) * lda + scalar_at(e));
             }
         }
         for (int idx = tid; idx < n * cb4; idx += blockDim.x) {
@@ -960,14 +1027,11 @@ state_scan_kernel(const float* __restrict__ rows, int64_t ld, int q_col, int k_c
             ks[dst] = act ? silu_(row[k_col + hq * d + j]) : row[k_col + hq * d + j];
             if (ROWS) as[dst] = aux[(t0 + c0 + c) * lda + aux_col + h * d + j];
         }
-        if (!ROWS) {
+        if (SCAL) {
             for (int c = tid; c < n; c += blockDim.x) {
-                const float* ar = aux + (t0 + c0 + c) * lda + aux_col;
-                as[c * 4 + 0] = ar[h];
-                if (MODE == 1) {
-                    as[c * 4 + 1] = ar[n_heads + h];
-                    as[c * 4 + 2] = ar[2 * n_heads + hq];
-                }
+                const float* ar = aux + (t0 + c0 + c) * lda;
+#pragma unroll
+                for (int e = SCAL0; e < SCAL1; e++) ss[c * 4 + e] = ar[scalar_at(e)];
             }
         }
         for (int idx = tid; idx < n * cb; idx += blockDim.x) {
@@ -995,11 +1059,12 @@ state_scan_kernel(const float* __restrict__ rows, int64_t ld, int q_col, int k_c
         const float* qb = qs + b * chunk * DPP;
         const float* kb = ks + b * chunk * DPP;
         const float* ab = as + b * chunk * a_tok;
+        const float* sb = ss + b * chunk * s_tok;
         const float* vb = vs + b * chunk * cb;
         ScanOperands<R, MODE> cur, nxt;
-        cur.load(qb, kb, ab, vb, 0, DPP, off, cb, col_l);
+        cur.load(qb, kb, ab, sb, vb, 0, DPP, off, cb, col_l);
         for (int c = 0; c < n; c++) {
-            if (c + 1 < n) nxt.load(qb, kb, ab, vb, c + 1, DPP, off, cb, col_l);
+            if (c + 1 < n) nxt.load(qb, kb, ab, sb, vb, c + 1, DPP, off, cb, col_l);
             const float o = scan_token<R, MODE>(S, cur, U);
             if (lk == 0 && live) raw_out[((t0 + c0 + c) * n_heads + h) * int64_t(dv) + col] = o;
             cur = nxt;
@@ -1101,15 +1166,19 @@ IB_EXPORT int ib_glu_act(const void* rows, int64_t ld, int64_t gate_col, int64_t
     return ib::check_launch("ib_glu_act");
 }
 
+// sigmoid 0: softmax scores, 1: sigmoid scores; group_best: how many of a group's largest scores are summed (1 or 2);
+// renormalise: the chosen scores are divided by their sum + sum_eps; mult: a constant on the weights.
 IB_EXPORT int ib_route(const float* logits, int64_t n_tokens, int n_experts, int top, int n_groups, int keep, float sum_eps,
-                       float* weights, int* chosen, cudaStream_t stream) {
+                       int sigmoid, int group_best, int renormalise, float mult, float* weights, int* chosen, cudaStream_t stream) {
     if (n_tokens <= 0) return IB_OK;
     if (n_experts <= 0 || n_groups <= 0 || n_experts % n_groups || keep <= 0 || keep > n_groups || top <= 0 ||
         top > keep * (n_experts / n_groups))
         return ib::fail(IB_ERR_ARG, "ib_route: %d experts in %d groups, %d kept, %d chosen", n_experts, n_groups, keep, top);
+    if (group_best != 1 && group_best != 2) return ib::fail(IB_ERR_ARG, "ib_route: a group's score is its largest or the sum of its two largest");
     const size_t smem = size_t(4) * (n_experts + n_groups) * sizeof(float);
     if (smem > 48 * 1024) return ib::fail(IB_ERR_ARG, "ib_route: %d experts do not fit", n_experts);
-    IB_LAUNCH(route_kernel, blocks_for(n_tokens, 4), 128, smem, logits, n_tokens, n_experts, top, n_groups, keep, sum_eps, weights, chosen);
+    IB_LAUNCH(route_kernel, blocks_for(n_tokens, 4), 128, smem, logits, n_tokens, n_experts, top, n_groups, keep, sum_eps,
+              sigmoid, group_best, renormalise, mult, weights, chosen);
     return ib::check_launch("ib_route");
 }
 
@@ -1205,16 +1274,19 @@ IB_EXPORT int ib_delta_prepare_max_dim() { return 32 * PREP_PER_LANE; }
 IB_EXPORT int ib_delta_prepare(const float* rows, int64_t ld, int col0, int a_col, int b_col, const float* filt_w, int taps,
                                float* tails, int inline_tail, const float* a_log, const float* dt_bias, float unit_eps, float q_scale,
                                const int* token_seg, const int* seg_start, const int* seg_slot, float* prep, int64_t ldp,
-                               int64_t n_tokens, int n_heads, int n_qk, int d, int dv, cudaStream_t stream) {
+                               int64_t n_tokens, int n_heads, int n_qk, int d, int dv, const float* z, int64_t ldz, int z_col,
+                               cudaStream_t stream) {
     if (n_tokens <= 0) return IB_OK;
     if (n_heads <= 0 || n_qk <= 0 || n_heads % n_qk || d <= 0 || dv <= 0 || d > 32 * PREP_PER_LANE)
         return ib::fail(IB_ERR_ARG, "ib_delta_prepare: %d heads on %d (q, k) heads of %d, values of %d", n_heads, n_qk, d, dv);
     if (filt_w && taps > 1 && !tails) return ib::fail(IB_ERR_ARG, "ib_delta_prepare: a filter of %d taps needs tails", taps);
-    if (ldp < 2 * int64_t(n_qk) * d + int64_t(n_heads) * dv + 2 * n_heads + n_qk) return ib::fail(IB_ERR_ARG, "ib_delta_prepare: prepared rows too short");
-    const int64_t warps = n_tokens * (n_qk + n_heads + 1);
+    const int64_t vec = 2 * int64_t(n_qk) * d + int64_t(n_heads) * dv;
+    if (ldp < (z ? (vec + 3) / 4 * 4 + int64_t(n_heads) * d : vec + n_heads) + n_heads + n_qk) return ib::fail(IB_ERR_ARG, "ib_delta_prepare: prepared rows too short");
+    const int64_t warps = n_tokens * (n_qk + n_heads + 1 + (z ? n_heads : 0));
     IB_LAUNCH(delta_prepare_kernel, blocks_for(warps, 4), 128, 0, rows, ld, col0, a_col, b_col, filt_w, filt_w ? taps : 0, tails,
               (filt_w && taps > 1) ? inline_tail : 0, a_log,
-              dt_bias, unit_eps, q_scale, token_seg, seg_start, seg_slot, prep, ldp, n_tokens, n_heads, n_qk, d, dv);
+              dt_bias, unit_eps, q_scale, token_seg, seg_start, seg_slot, prep, ldp, n_tokens, n_heads, n_qk, d, dv,
+              z, ldz, z_col);
     return ib::check_launch("ib_delta_prepare");
 }
 
@@ -1234,26 +1306,27 @@ template <int R, int MODE>
 static int launch_scan(dim3 grid, int threads, size_t smem, cudaStream_t stream, const float* rows, int64_t ld, int q_col,
                        int k_col, int v_col, const float* aux, int64_t lda, int aux_col, float* state, const int* seg_start,
                        const int* seg_slot, float* raw_out, int n_heads, int hpq, int d, int dv, int cb, int chunk, int write_state,
-                       int pipelined, const float* bonus, int act) {
+                       int pipelined, const float* bonus, int act, int scal_col) {
     IB_LAUNCH((state_scan_kernel<R, MODE>), grid, threads, smem, rows, ld, q_col, k_col, v_col, aux, lda, aux_col, state, seg_start,
-              seg_slot, raw_out, n_heads, hpq, d, dv, cb, chunk, write_state, pipelined, bonus, act);
+              seg_slot, raw_out, n_heads, hpq, d, dv, cb, chunk, write_state, pipelined, bonus, act, scal_col);
     return ib::check_launch("ib_state_scan");
 }
 
 // mode 0: a decay per key channel (aux: decays at aux_col + h d); mode 1: gated delta rule (aux: g, beta, k.q);
 // mode 2: a decay per head (aux: at aux_col + h; lda 0: the same for every token); mode 3: as mode 0 with the read-out
-// before the write and `bonus` [heads, d] on the current token.
+// before the write and `bonus` [heads, d] on the current token; mode 4: delta rule with decays as mode 0 and beta, k.q at
+// scal_col of the aux rows.
 // `spread` (prompt portions): a head's columns go to more, smaller CTAs until there is about one per SM (sm_count).
 IB_EXPORT int ib_state_scan(int mode, const float* rows, int64_t ld, int q_col, int k_col, int v_col, const float* aux,
                             int64_t lda, int aux_col, float* state, const int* seg_start, const int* seg_slot,
                             float* raw_out, int n_segments, int n_heads, int heads_per_qk, int d, int dv, int write_state,
-                            int spread, int sm_count, cudaStream_t stream, const float* bonus, int act) {
+                            int spread, int sm_count, cudaStream_t stream, const float* bonus, int act, int scal_col) {
     if (n_segments <= 0) return IB_OK;
     if (n_heads <= 0 || n_heads > 65535 || heads_per_qk <= 0 || n_heads % heads_per_qk || d <= 0 || dv <= 0 || d > LK * 32)
         return ib::fail(IB_ERR_ARG, "ib_state_scan: %d heads with a state of %d x %d do not fit", n_heads, d, dv);
-    if (mode < 0 || mode > 3) return ib::fail(IB_ERR_ARG, "ib_state_scan: unknown mode %d", mode);
+    if (mode < 0 || mode > 4) return ib::fail(IB_ERR_ARG, "ib_state_scan: unknown mode %d", mode);
     if (mode == 3 && !bonus) return ib::fail(IB_ERR_ARG, "ib_state_scan: mode 3 needs the bonus");
-    const bool decay_rows = mode == 0 || mode == 3;
+    const bool decay_rows = mode == 0 || mode == 3 || mode == 4;
     const int r = d <= 32 ? 4 : (d <= 64 ? 8 : (d <= 128 ? 16 : 32));
     int cb = 32;
     while (cb > 4 && cb / 2 >= dv) cb /= 2;                     // no CTA wider than the head
@@ -1268,7 +1341,7 @@ IB_EXPORT int ib_state_scan(int mode, const float* rows, int64_t ld, int q_col, 
                           v_col % 4 == 0 && (!decay_rows || (lda % 4 == 0 && aux_col % 4 == 0 && !(uintptr_t(aux) & 15))) &&
                           !(uintptr_t(rows) & 15);
     const int dpp = LK * (r + 4), n_buf = pipelined ? 2 : 1;
-    const int per_token = 2 * dpp + (decay_rows ? dpp : 4) + cb;
+    const int per_token = 2 * dpp + (decay_rows ? dpp : 4) + (mode == 4 ? 4 : 0) + cb;
     int chunk = 11264 / (n_buf * per_token);
     chunk = chunk < 1 ? 1 : (chunk > 16 ? 16 : chunk);
     const size_t smem = size_t(n_buf) * chunk * per_token * sizeof(float);
@@ -1277,7 +1350,13 @@ IB_EXPORT int ib_state_scan(int mode, const float* rows, int64_t ld, int q_col, 
     const int threads = cb * LK;
 #define IB_SCAN(RR, MM)                                                                                                          \
     return launch_scan<RR, MM>(grid, threads, smem, stream, rows, ld, q_col, k_col, v_col, aux, lda, aux_col, state, seg_start, \
-                               seg_slot, raw_out, n_heads, heads_per_qk, d, dv, cb, chunk, write_state, pipelined, bonus, act)
+                               seg_slot, raw_out, n_heads, heads_per_qk, d, dv, cb, chunk, write_state, pipelined, bonus, act, scal_col)
+    if (mode == 4) {
+        if (r == 4) IB_SCAN(4, 4);
+        if (r == 8) IB_SCAN(8, 4);
+        if (r == 16) IB_SCAN(16, 4);
+        IB_SCAN(32, 4);
+    }
     if (mode == 2) {
         if (r == 4) IB_SCAN(4, 2);
         if (r == 8) IB_SCAN(8, 2);

@@ -26,6 +26,7 @@ class Model:
         self.embedding = self._build_part("embedding", spec.embedding, weights)
         self.blocks: List[Block] = [self._build_block(ls, weights) for ls in spec.layers]
         self.final_norm = self._build_part("norm", spec.final_norm, weights)
+        self.stream = self._build_part("stream", spec.stream, weights) if spec.stream is not None else None
         self.head = self._build_part("head", spec.head, weights)
         self.head.tie(self.embedding)
 
@@ -44,6 +45,8 @@ class Model:
         for b in self.blocks:
             yield from b.parts.values()
         yield self.final_norm
+        if self.stream is not None:
+            yield self.stream
         yield self.head
 
     def graph_safe(self) -> bool:
@@ -63,11 +66,16 @@ class Model:
 
     def forward(self, step, cache_views: Mapping[int, object]) -> torch.Tensor:
         h = self.embedding.forward(step)                                           # float32 [T, hidden]
+        if self.stream is not None:
+            h = self.stream.open(h)
         for call in self.spec.schedule:
             h = self.blocks[call.layer].forward(h, step, cache_views[call.cache], call.write_cache)
         if step.n_want == 0:
-            return torch.empty((0, self.spec.vocab_size), dtype=torch.float32, device=h.device)
-        normed = self.final_norm.forward(h, rows=step.want_rows)                  # [wanted, hidden]
+            return torch.empty((0, self.spec.vocab_size), dtype=torch.float32, device=self.rt.device)
+        if self.stream is not None:
+            normed = self.stream.close(h, self.final_norm, step.want_rows)
+        else:
+            normed = self.final_norm.forward(h, rows=step.want_rows)              # [wanted, hidden]
         return self.head.forward(normed)                                           # float32 [wanted, vocab]
 
     def weight_bytes(self) -> int:

@@ -550,17 +550,20 @@ def glu_act(rows: torch.Tensor, gate_col: int, up_col: int, width: int, kind: st
     return out
 
 
-def route(logits: torch.Tensor, top: int, n_groups: int = 1, keep: int = 1, sum_eps: float = 0.0, want_chosen: bool = False):
-    """Router of a mixture of experts on float32 logits [T, E]: softmax over all experts; the ``keep`` groups (of
-    E / n_groups neighbouring experts) with the largest single score stay; of their experts the ``top`` largest are
-    chosen; weights are scores / (their sum + sum_eps). Returns (weights float32 [T, E], zero where not chosen;
-    chosen int32 [T, top] or None)."""
+def route(logits: torch.Tensor, top: int, n_groups: int = 1, keep: int = 1, sum_eps: float = 0.0, want_chosen: bool = False,
+          sigmoid: bool = False, group_best: int = 1, renormalise: bool = True, mult: float = 1.0):
+    """Router of a mixture of experts on float32 logits [T, E]: softmax over all experts (``sigmoid``: each logit's
+    sigmoid); the ``keep`` groups (of E / n_groups neighbouring experts) with the largest score stay, a group's score
+    being its largest (``group_best`` 2: the sum of its two largest); of their experts the ``top`` largest are chosen;
+    weights are scores / (their sum + sum_eps) (not ``renormalise``: the scores as they are), times ``mult``. Returns
+    (weights float32 [T, E], zero where not chosen; chosen int32 [T, top] or None)."""
     _check(logits, "logits", torch.float32)
     T, E = logits.shape
     weights = torch.empty((T, E), dtype=torch.float32, device=logits.device)
     chosen = torch.empty((T, top), dtype=torch.int32, device=logits.device) if want_chosen else None
-    f = _fn("mix", "ib_route", [c_void_p, c_int64, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p])
-    _call(f, logits.data_ptr(), T, E, int(top), int(n_groups), int(keep), float(sum_eps), weights.data_ptr(), _ptr(chosen), _stream())
+    f = _fn("mix", "ib_route", [c_void_p, c_int64, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p])
+    _call(f, logits.data_ptr(), T, E, int(top), int(n_groups), int(keep), float(sum_eps), int(bool(sigmoid)), int(group_best),
+          int(bool(renormalise)), float(mult), weights.data_ptr(), _ptr(chosen), _stream())
     return weights, chosen
 
 
@@ -696,17 +699,34 @@ def state_scan_max_dim() -> int:
     return int(_fn("mix", "ib_state_scan_max_dim", [])())
 
 
+def delta_columns(n_heads: int, n_qk: int, dim: int, v_dim: int, per_channel: bool):
+    """(first column of the decays, first column of [beta | k.q]) in the rows that ``delta_prepare`` returns."""
+    C = 2 * n_qk * dim + n_heads * v_dim
+    if per_channel:
+        C = (C + 3) // 4 * 4
+    return C, C + (n_heads * dim if per_channel else n_heads)
+
+
 def delta_prepare(rows: torch.Tensor, col0: int, a_col: int, b_col: int, filt_w: Optional[torch.Tensor],
                   tails: Optional[torch.Tensor], a_log: torch.Tensor, dt_bias: torch.Tensor, unit_eps: float, q_scale: float,
-                  step, n_heads: int, n_qk: int, dim: int, v_dim: int, inline_tail: bool = False) -> torch.Tensor:
+                  step, n_heads: int, n_qk: int, dim: int, v_dim: int, inline_tail: bool = False, decay_rows: Optional[torch.Tensor] = None,
+                  decay_col: int = 0) -> torch.Tensor:
     """What the gated delta rule reads, from float32 projected rows [.. q (n_qk x dim) | k | v (n_heads x v_dim) ..]
     (from column col0; per-head step-size logits at a_col, write-strength logits at b_col): every q, k, v channel
     through its causal filter (``filt_w`` float32 [taps, channels], ``tails`` float32 [slots, taps - 1, channels]) and
     silu; q and k made unit vectors per head, q times q_scale. Returns float32 [T, q | k | v | g | beta | k.q].
-    ``inline_tail`` (only for steps of one token per request): the kernel also moves the tails (no ``tail_update``)."""
+    ``inline_tail`` (only for steps of one token per request): the kernel also moves the tails (no ``tail_update``).
+    With ``decay_rows`` (float32 rows of n_heads x dim logits from column ``decay_col``) the decay is a number per head
+    and key channel (dt_bias [n_heads * dim]) and the result is [q | k | v | up to a multiple of 4 | g (n_heads x dim) |
+    beta | k.q]; see ``delta_columns``."""
     _check(rows, "rows", torch.float32)
     T, ld = rows.shape
     C = 2 * n_qk * dim + n_heads * v_dim
+    if decay_rows is not None:
+        a_col = 0
+        _check(decay_rows, "decay_rows", torch.float32)
+        if decay_rows.shape[0] != T or decay_col < 0 or decay_col + n_heads * dim > decay_rows.shape[1]:
+            raise KernelError("delta_prepare: the decay logits lie outside their rows")
     if col0 + C > ld or a_col + n_heads > ld or b_col + n_heads > ld:
         raise KernelError("delta_prepare: columns lie outside the rows")
     taps = 0
@@ -720,14 +740,16 @@ def delta_prepare(rows: torch.Tensor, col0: int, a_col: int, b_col: int, filt_w:
             if tuple(tails.shape[1:]) != (taps - 1, C):
                 raise KernelError(f"tails must be [slots, {taps - 1}, {C}], got {tuple(tails.shape)}")
     _check(a_log, "a_log", torch.float32, (n_heads,))
-    _check(dt_bias, "dt_bias", torch.float32, (n_heads,))
-    ldp = (C + 2 * n_heads + n_qk + 3) // 4 * 4
+    _check(dt_bias, "dt_bias", torch.float32, (n_heads if decay_rows is None else n_heads * dim,))
+    ldp = (delta_columns(n_heads, n_qk, dim, v_dim, decay_rows is not None)[1] + n_heads + n_qk + 3) // 4 * 4
     prep = torch.empty((T, ldp), dtype=torch.float32, device=rows.device)
     f = _fn("mix", "ib_delta_prepare", [c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float,
-                                        c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int64, c_int, c_int, c_int, c_int, c_void_p])
+                                        c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int64, c_int, c_int, c_int, c_int, c_void_p, c_int64,
+                                        c_int, c_void_p])
     _call(f, rows.data_ptr(), ld, int(col0), int(a_col), int(b_col), _ptr(filt_w), taps, _ptr(tails) if taps > 1 else None,
           int(bool(inline_tail)), a_log.data_ptr(), dt_bias.data_ptr(), float(unit_eps), float(q_scale), step.token_seg.data_ptr(), step.seg_start.data_ptr(),
-          step.seg_slot.data_ptr(), prep.data_ptr(), ldp, T, n_heads, n_qk, dim, v_dim, _stream())
+          step.seg_slot.data_ptr(), prep.data_ptr(), ldp, T, n_heads, n_qk, dim, v_dim, _ptr(decay_rows),
+          0 if decay_rows is None else decay_rows.shape[1], int(decay_col), _stream())
     return prep
 
 
@@ -742,21 +764,23 @@ def tail_update(rows: torch.Tensor, col0: int, tails: torch.Tensor, seg_start: t
           seg_slot.numel(), _stream())
 
 
-SCAN_ROW_DECAY, SCAN_DELTA_RULE, SCAN_HEAD_DECAY, SCAN_BONUS = 0, 1, 2, 3
+SCAN_ROW_DECAY, SCAN_DELTA_RULE, SCAN_HEAD_DECAY, SCAN_BONUS, SCAN_CHANNEL_DELTA = 0, 1, 2, 3, 4
 SCAN_SPREAD_FROM = 8          # segments of more tokens than this spread a head's columns over more CTAs
 
 
 def state_scan(mode: int, rows: torch.Tensor, q_col: int, k_col: int, v_col: int, aux: torch.Tensor, aux_col: int,
                state: torch.Tensor, seg_start: torch.Tensor, seg_slot: torch.Tensor, n_heads: int, heads_per_qk: int,
                dim: int, v_dim: int, write_state: bool = True, max_len: int = 1, bonus: Optional[torch.Tensor] = None,
-               silu: bool = False) -> torch.Tensor:
+               silu: bool = False, scalar_col: int = 0) -> torch.Tensor:
     """A linear recurrence with a float32 matrix state [slots, heads, dim, v_dim], over the tokens of every segment
     in order. SCAN_ROW_DECAY: S <- diag(a) S + k v^T, o = S^T q, with a in ``aux`` columns aux_col + h * dim.
     SCAN_DELTA_RULE: S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q, with ``aux`` columns [g (heads) | beta
     (heads) | k.q (heads / heads_per_qk)] from aux_col. q, k at q_col, k_col + (h // heads_per_qk) * dim and v at
     v_col + h * v_dim of the float32 ``rows``. SCAN_HEAD_DECAY: S <- g_h S + k v^T, o = S^T q, with ``aux`` float32
     [heads] (a constant per head) or [T, ...] with g at column aux_col + h. SCAN_BONUS: o = (S + diag(u) k v^T)^T q, then
-    S <- diag(a) S + k v^T, with a as for SCAN_ROW_DECAY and u = ``bonus`` float32 [heads, dim].
+    S <- diag(a) S + k v^T, with a as for SCAN_ROW_DECAY and u = ``bonus`` float32 [heads, dim]. SCAN_CHANNEL_DELTA:
+    S <- diag(a) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q, with a as for SCAN_ROW_DECAY and ``aux`` columns
+    [beta (heads) | k.q (heads / heads_per_qk)] from ``scalar_col``.
     ``silu``: q, k and v are z * sigmoid(z) of what the rows hold (applied while the tokens are staged).
     Returns o float32 [T, heads * v_dim]."""
     _check(rows, "rows", torch.float32)
@@ -786,7 +810,10 @@ def state_scan(mode: int, rows: torch.Tensor, q_col: int, k_col: int, v_col: int
         if aux_col + n_heads > aux.shape[0]:
             raise KernelError("a decay per head needs one value per head")
     else:
-        need = {SCAN_ROW_DECAY: n_heads * dim, SCAN_BONUS: n_heads * dim, SCAN_DELTA_RULE: 2 * n_heads + n_qk, SCAN_HEAD_DECAY: n_heads}[mode]
+        need = {SCAN_ROW_DECAY: n_heads * dim, SCAN_BONUS: n_heads * dim, SCAN_DELTA_RULE: 2 * n_heads + n_qk, SCAN_HEAD_DECAY: n_heads,
+                SCAN_CHANNEL_DELTA: n_heads * dim}[mode]
+        if mode == SCAN_CHANNEL_DELTA and (aux.dim() != 2 or scalar_col < 0 or scalar_col + n_heads + n_qk > aux.shape[1]):
+            raise KernelError("the write strengths lie outside their rows")
         if aux.dim() != 2 or aux.shape[0] != T or aux_col + need > aux.shape[1]:
             raise KernelError("the decay columns lie outside their rows")
         lda = aux.shape[1]
@@ -800,10 +827,11 @@ def state_scan(mode: int, rows: torch.Tensor, q_col: int, k_col: int, v_col: int
     spread = int(max_len) >= SCAN_SPREAD_FROM
     sm_count = torch.cuda.get_device_properties(rows.device).multi_processor_count if spread else 0
     f = _fn("mix", "ib_state_scan", [c_int, c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_int64, c_int, c_void_p, c_void_p,
-                                     c_void_p, c_void_p] + [c_int] * 8 + [c_void_p, c_void_p, c_int])
+                                     c_void_p, c_void_p] + [c_int] * 8 + [c_void_p, c_void_p, c_int, c_int])
     _call(f, int(mode), rows.data_ptr(), ld, int(q_col), int(k_col), int(v_col), aux.data_ptr(), lda, int(aux_col),
           state.data_ptr(), seg_start.data_ptr(), seg_slot.data_ptr(), out.data_ptr(), S, n_heads, int(heads_per_qk), dim, v_dim,
-          int(write_state), int(spread), sm_count, _stream(), _ptr(bonus) if mode == SCAN_BONUS else None, int(bool(silu)))
+          int(write_state), int(spread), sm_count, _stream(), _ptr(bonus) if mode == SCAN_BONUS else None, int(bool(silu)),
+          int(scalar_col))
     return out
 
 
@@ -1263,4 +1291,129 @@ def relu_sq(x: torch.Tensor, col0: int = 0, width: Optional[int] = None) -> torc
     out = torch.empty((T, width), dtype=x.dtype, device=x.device)
     f = _fn("post", "ib_relu_sq", [c_void_p, c_int64, c_int64, c_int64, c_void_p, c_int64, c_int, c_void_p])
     _call(f, x.data_ptr(), ld, int(col0), width, out.data_ptr(), T, dtype_code(x.dtype), _stream())
+    return out
+
+
+# ----------------------------------------------------------------------------- several residual streams, sinusoidal positions
+
+def embedding_sinusoid(table: torch.Tensor, ids: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor,
+                       status: Optional[torch.Tensor] = None, feedback: Optional[torch.Tensor] = None,
+                       token_seg: Optional[torch.Tensor] = None, seg_slot: Optional[torch.Tensor] = None,
+                       scale: float = 1.0) -> torch.Tensor:
+    """``embedding`` plus a position vector: channels 2i and 2i + 1 of token t take sin and cos of positions[t] * freq[i]
+    (``freq`` float64 [ceil(width / 2)])."""
+    _check(table, "table")
+    _check(ids, "ids", torch.int32)
+    T, (V, W) = ids.numel(), table.shape
+    _check(positions, "positions", torch.int32, (T,))
+    _check(freq, "freq", torch.float64, ((W + 1) // 2,))
+    out = torch.empty((T, W), dtype=torch.float32, device=table.device)
+    if feedback is not None:
+        _check(feedback, "feedback", torch.int32)
+        _check(token_seg, "token_seg", torch.int32, (T,))
+        _check(seg_slot, "seg_slot", torch.int32)
+    f = _fn("stream", "ib_embedding_sinusoid", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int64, c_int64, c_int64] +
+            [c_void_p] * 5 + [c_float, c_void_p])
+    _call(f, table.data_ptr(), dtype_code(table.dtype), ids.data_ptr(), positions.data_ptr(), freq.data_ptr(), T, W, V, out.data_ptr(),
+          _ptr(status), _ptr(feedback), _ptr(token_seg), _ptr(seg_slot), float(scale), _stream())
+    return out
+
+
+def stream_link_max_streams() -> int:
+    return int(_fn("stream", "ib_stream_link_max_streams", [])())
+
+
+def stream_link(x: torch.Tensor, n_streams: int, out_dtype: torch.dtype, y: Optional[torch.Tensor] = None,
+                mix: Optional[torch.Tensor] = None, out_w: Optional[torch.Tensor] = None, in_w: Optional[torch.Tensor] = None,
+                norm_w: Optional[torch.Tensor] = None, eps: float = 0.0, groups: int = 1, store: bool = True,
+                rows: Optional[torch.Tensor] = None):
+    """``n_streams`` residual streams x float32 [T, n, W] ([T, W]: all n are this row) first take a sublayer's result y
+    float32 [T, W]: x_t <- sum_s mix[s, t] x_s + out_w[t] y (y None: they stay), which with ``store`` is kept, over x
+    where x holds all streams and in a new tensor where it holds one row; then their combination u = sum_s in_w[s] x_s
+    (None: the plain sum) is normalised in ``groups`` equal parts, part / sqrt(mean(part^2) + eps), times norm_w [W]
+    (None: u itself). ``rows`` (int32) picks and orders tokens (nothing is stored then). Returns (streams or x,
+    the normalised rows in ``out_dtype``)."""
+    _check(x, "x", torch.float32)
+    shared = x.dim() == 2
+    T, W = x.shape[0], x.shape[-1]
+    n = int(n_streams)
+    if not shared:
+        _check(x, "x", None, (T, n, W))
+    if y is not None:
+        _check(y, "y", torch.float32, (T, W))
+        _check(mix, "mix", torch.float32, (n, n))
+        _check(out_w, "out_w", torch.float32, (n,))
+    if in_w is not None:
+        _check(in_w, "in_w", torch.float32, (n,))
+    if norm_w is not None:
+        _check(norm_w, "norm_w", torch.float32, (W,))
+    n_rows = T
+    if rows is not None:
+        _check(rows, "rows", torch.int32)
+        n_rows, store = rows.numel(), False
+    out_x = None
+    if store and y is not None:
+        out_x = torch.empty((T, n, W), dtype=torch.float32, device=x.device) if shared and n > 1 else x
+    out = torch.empty((n_rows, W), dtype=out_dtype, device=x.device)
+    f = _fn("stream", "ib_stream_link", [c_void_p, c_int64, c_int64] + [c_void_p] * 5 + [c_float, c_int, c_int64, c_void_p, c_void_p, c_int,
+                                         c_void_p, c_int64, c_int, c_void_p])
+    _call(f, x.data_ptr(), W if shared else n * W, 0 if shared else W, _ptr(y), _ptr(mix) if y is not None else None,
+          _ptr(out_w) if y is not None else None, _ptr(in_w), _ptr(norm_w), float(eps), int(groups), W, _ptr(out_x), out.data_ptr(),
+          dtype_code(out_dtype), _ptr(rows), n_rows, n, _stream())
+    return (out_x if out_x is not None else x), out
+
+
+# ----------------------------------------------------------------------------- attention whose heads exchange their scores
+
+def kv_store(rows: torch.Tensor, k_col: int, v_col: int, step, block_table: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+             n_kv: int, head_dim: int, v_head_dim: int) -> None:
+    """Keys and values of projected rows (from columns k_col and v_col) into the tokens' pages, as they are."""
+    _check(rows, "rows")
+    T, ld = rows.shape
+    n_pages, ckv, page_size, _ = k_cache.shape
+    _check(k_cache, "k_cache", rows.dtype, (n_pages, n_kv, page_size, head_dim))
+    _check(v_cache, "v_cache", rows.dtype, (n_pages, n_kv, page_size, v_head_dim))
+    if min(k_col, v_col) < 0 or k_col + n_kv * head_dim > ld or v_col + n_kv * v_head_dim > ld:
+        raise KernelError("k and v lie outside the rows")
+    _check(block_table, "block_table", torch.int32)
+    f = _fn("talk", "ib_kv_store", [c_void_p, c_int64, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_int64] +
+            [c_int] * 4 + [c_int64, c_int, c_void_p, c_void_p])
+    _call(f, rows.data_ptr(), ld, int(k_col), int(v_col), step.positions.data_ptr(), step.token_seg.data_ptr(), block_table.data_ptr(),
+          block_table.shape[1], k_cache.data_ptr(), v_cache.data_ptr(), T, n_kv, head_dim, v_head_dim, page_size, n_pages,
+          dtype_code(rows.dtype), _ptr(step.status), _stream())
+
+
+def talk_attention_fits(n_heads: int, head_dim: int, v_head_dim: int) -> bool:
+    return bool(_fn("talk", "ib_talk_attention_fits", [c_int, c_int, c_int])(int(n_heads), int(head_dim), int(v_head_dim)))
+
+
+def _check_talk(q, q_col, k_cache, v_cache, block_table, n_heads, n_kv, head_dim, v_head_dim, talk):
+    _check(q, "q")
+    T, ld = q.shape
+    if q_col < 0 or q_col + n_heads * head_dim > ld:
+        raise KernelError("the queries lie outside their rows")
+    n_pages, ckv, page_size, _ = k_cache.shape
+    _check(k_cache, "k_cache", q.dtype, (n_pages, n_kv, page_size, head_dim))
+    _check(v_cache, "v_cache", q.dtype, (n_pages, n_kv, page_size, v_head_dim))
+    _check(block_table, "block_table", torch.int32)
+    if talk is not None:
+        _check(talk, "talk", torch.float32, (n_heads, n_heads))
+    return T, ld, n_pages, page_size
+
+
+def talk_attention(q: torch.Tensor, q_col: int, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor, step,
+                   n_heads: int, n_kv: int, head_dim: int, v_head_dim: int, window: Optional[int], chunk: Optional[int], scale: float,
+                   cap: float, talk: Optional[torch.Tensor]) -> torch.Tensor:
+    """Causal attention of every token over its request's pages, queries from column ``q_col`` of the rows q -> [T, heads *
+    v_head_dim]. Scores are capped (``cap`` * tanh(score / cap); 0: not), then exchanged among the heads (``talk`` float32
+    [heads, heads]: score_h <- sum_g talk[h, g] score_g; None: not). A query sees the keys of its own chunk of ``chunk``
+    positions (and of ``window``) only."""
+    T, ld, n_pages, page_size = _check_talk(q, q_col, k_cache, v_cache, block_table, n_heads, n_kv, head_dim, v_head_dim, talk)
+    out = torch.empty((T, n_heads * v_head_dim), dtype=q.dtype, device=q.device)
+    f = _fn("talk", "ib_talk_attention", [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int64] +
+            [c_int] * 7 + [c_float, c_float, c_void_p, c_int64, c_int, c_void_p, c_void_p])
+    _call(f, q.data_ptr() + q_col * q.element_size(), ld, k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(),
+          block_table.shape[1], step.token_seg.data_ptr(), step.positions.data_ptr(), out.data_ptr(), T, n_heads, n_kv, head_dim,
+          v_head_dim, page_size, int(window or 0), int(chunk or 0), float(scale), float(cap or 0.0), _ptr(talk), n_pages,
+          dtype_code(q.dtype), _ptr(step.status), _stream())
     return out

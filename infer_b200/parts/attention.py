@@ -40,6 +40,14 @@ fills the pages (``head_prepare``), then through the attention kernels that take
 ``channel_gate``       the joined heads are multiplied, channel by channel, by sigmoid(x Wg^T) (role gate,
                        [heads * v_head_dim, hidden]) before the output product; Wg rides in the q/k/v product
 ``sink``               as above
+
+A fourth group goes through kernels that work on all heads of a (query, key) pair at once:
+
+``score_cap``          the scaled score s becomes cap * tanh(s / cap)
+``head_exchange``      then score_h <- sum_g T[h, g] score_g with a learned matrix T (role talk, [heads, heads]), before mask
+                       and softmax
+``chunk``              query i sees key j <= i only if floor(i / chunk) = floor(j / chunk); pages of past chunks go back
+``o_bias``             a bias on the output product (role o_bias)
 """
 from __future__ import annotations
 
@@ -56,7 +64,8 @@ from .linear import Linear
 _NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
           "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias",
           "q_filter": "q_proj.filter", "k_filter": "k_proj.filter", "v_filter": "v_proj.filter", "gate": "gate_proj.weight",
-          "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "rel": "distance_bias.weight", "sink": "sinks"}
+          "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "rel": "distance_bias.weight", "sink": "sinks",
+          "talk": "head_exchange.weight", "o_bias": "o_proj.bias"}
 
 
 def _names(spec: PartSpec):
@@ -132,7 +141,14 @@ class Attention(Mixer):
                          or self.values_are_keys or self.channel_gate)
         if self.per_head:
             self._check_per_head(spec)
-        own_path = self.per_head or spec.get("qk_row_norm_eps") is not None or spec.get("distance_bias") is not None or bool(spec.get("sink", False))
+        self.cap = float(spec.get("score_cap") or 0.0)
+        self.exchange = bool(spec.get("head_exchange", False))
+        self.chunk = int(spec["chunk"]) if spec.get("chunk") is not None else None
+        self.all_heads = self.cap != 0.0 or self.exchange or self.chunk is not None
+        self.has_o_bias = bool(spec.get("o_bias", False))
+        if self.all_heads:
+            self._check_all_heads(spec)
+        own_path = self.per_head or self.all_heads or spec.get("qk_row_norm_eps") is not None or spec.get("distance_bias") is not None or bool(spec.get("sink", False))
         if self.prepared and not own_path:
             if max(self.head_dim, self.v_dim) > ops.qkv_prepare_max_head_dim():
                 raise ValueError(f"the prepare kernel takes head sizes up to {ops.qkv_prepare_max_head_dim()}, "
@@ -143,7 +159,8 @@ class Attention(Mixer):
         self.distance_bias = spec.get("distance_bias")
         self.has_sink = bool(spec.get("sink", False))
         self.row_norm = self.row_norm_eps is not None
-        if self.per_head:
+        self.talk_w = None
+        if self.per_head or self.all_heads:
             self.prepared = self.biased = False
         elif self.row_norm or self.distance_bias is not None or self.has_sink:
             # these scores are not the ones the fast kernels compute; the projected rows go through the row-norm kernel
@@ -179,6 +196,16 @@ class Attention(Mixer):
         if self.values_are_keys and self.v_dim != self.head_dim:
             raise ValueError("values that are the keys have the keys' size")
 
+    def _check_all_heads(self, spec):
+        if self.cap < 0 or (self.chunk is not None and self.chunk <= 0):
+            raise ValueError("score_cap and chunk must be positive (or absent)")
+        if self.per_head or self.taps > 0 or self.value_norm_eps is not None or self.head_gate or self.position is not None \
+                or spec.get("qk_row_norm_eps") is not None or spec.get("distance_bias") is not None or spec.get("sink", False):
+            raise ValueError("capped or exchanged scores and chunks do not combine with rotation, norms, filters, gates, biases by "
+                             "distance or sinks")
+        if not ops.talk_attention_fits(self.n_heads, self.head_dim, self.v_dim):
+            raise ValueError(f"{self.n_heads} heads of {self.head_dim} / {self.v_dim} are beyond what the kernels that exchange scores hold")
+
     @classmethod
     def param_shapes(cls, spec):
         H, nh, nkv, hd = int(spec["hidden_size"]), int(spec["num_heads"]), int(spec["num_kv_heads"]), int(spec["head_dim"])
@@ -205,6 +232,10 @@ class Attention(Mixer):
             shapes[n["rel"]] = (int(db["buckets"]) if db.get("buckets") is not None else -1, nh)
         if spec.get("sink", False):
             shapes[n["sink"]] = (nh,)
+        if spec.get("head_exchange", False):
+            shapes[n["talk"]] = (nh, nh)
+        if spec.get("o_bias", False):
+            shapes[n["o_bias"]] = (H,)
         return shapes
 
     @classmethod
@@ -219,6 +250,8 @@ class Attention(Mixer):
             return 1.0 + 0.1 * torch.randn(shape, generator=gen, dtype=torch.float32, device=gen.device)
         if name in (n["rel"], n["sink"]):
             return torch.randn(shape, generator=gen, dtype=torch.float32, device=gen.device)
+        if name == n["talk"]:
+            return torch.eye(shape[0], device=gen.device) + 0.3 * torch.randn(shape, generator=gen, dtype=torch.float32, device=gen.device)
         return super().init_params(spec, name, shape, gen)
 
     def load(self, params):
@@ -236,10 +269,12 @@ class Attention(Mixer):
             if w.shape[0] > b.numel():
                 b = torch.cat([b, torch.zeros(w.shape[0] - b.numel(), device=b.device)])
         self.qkv = Linear(self.rt, w, b)
-        self.o = Linear(self.rt, params[n["o"]])
+        self.o = Linear(self.rt, params[n["o"]], params[n["o_bias"]].float() if self.has_o_bias else None)
         f32 = dict(device=self.rt.device, dtype=torch.float32)
         if self.head_norm_eps is not None:
             self.q_norm_w, self.k_norm_w = params[n["q_norm"]].to(**f32).contiguous(), params[n["k_norm"]].to(**f32).contiguous()
+        if self.exchange:
+            self.talk_w = params[n["talk"]].to(**f32).contiguous()
         if self.slopes is not None:
             self.slopes_w = torch.tensor(self.slopes, **f32)
         if self.row_norm:
@@ -257,7 +292,7 @@ class Attention(Mixer):
 
     def cache_need(self):
         pages = PagedKVNeed(self.n_kv, self.head_dim, self.window, None if self.v_dim == self.head_dim else self.v_dim,
-                            keep_first=self.keep_first if self.window is not None else 0)
+                            keep_first=self.keep_first if self.window is not None else 0, chunk=self.chunk)
         if self.taps > 1:
             # the last taps - 1 projected rows of the request, in the compute dtype (copies, not sums)
             return CompositeNeed({"pages": pages, "tails": StateNeed({"qkv": ((self.taps - 1, self.n_qkv), None)})})
@@ -281,7 +316,7 @@ class Attention(Mixer):
     def input_product(self):
         """The q/k/v(/gate) product, for a block that joins the products of parts reading the same rows. Only the
         prepared path reads its rows by (leading dimension, first column)."""
-        return (self.qkv, "compute") if (self.prepared or self.biased or self.per_head) else None
+        return (self.qkv, "compute") if (self.prepared or self.biased or self.per_head or self.all_heads) else None
 
     def drop_input_product(self):
         self.qkv = None
@@ -333,7 +368,21 @@ class Attention(Mixer):
             ops.gate_mul(ctx, qkv, col0 + self.n_qkv)
         return self._project_out(ctx, residual)
 
+    def _forward_all_heads(self, qkv, col0, step, cache, residual, write_cache):
+        """Capped scores, the exchange among the heads and chunks. The part's columns [q | k | v] start at ``col0``; keys
+        and values go to the pages as projected, the attention kernels read the queries where they are."""
+        table = step.block_tables[cache.group]
+        nq, nk = self.n_heads * self.head_dim, self.n_kv * self.head_dim
+        if write_cache:
+            ops.kv_store(qkv, col0 + nq, col0 + nq + nk, step, table, cache.k, cache.v, self.n_kv, self.head_dim, self.v_dim)
+        ctx = ops.talk_attention(qkv, col0, cache.k, cache.v, table, step, self.n_heads, self.n_kv, self.head_dim, self.v_dim, self.window,
+                                 self.chunk, self.scale, self.cap, self.talk_w)
+        return self._project_out(ctx, residual)
+
     def forward(self, x, step, cache, residual, write_cache=True):
+        if self.all_heads:
+            qkv, col0 = own_or_projected(self, x, self.qkv)
+            return self._forward_all_heads(qkv, col0, step, cache, residual, write_cache)
         if self.per_head:
             qkv, col0 = own_or_projected(self, x, self.qkv)
             return self._forward_per_head(qkv, col0, step, cache, residual, write_cache)

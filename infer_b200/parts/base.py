@@ -31,6 +31,7 @@ class PagedKVNeed:
                                       # row per position serves both, as in attention through a shared latent); there
                                       # are no value pages and the view's ``v`` is None
     keep_first: int = 0               # with a window: the positions below this stay readable for every later query
+    chunk: Optional[int] = None       # n: a query reads keys of its own chunk of n positions only (counted from position 0)
 
     @property
     def value_dim(self) -> int:
@@ -194,6 +195,23 @@ class Gate(Part):
         raise NotImplementedError
 
 
+class Connection(Part):
+    """How one sublayer reads from and writes to a residual stream that is more than one row per token."""
+
+
+class Stream(Part):
+    """The residual stream of a model whose blocks pass on something else than float32 rows [T, hidden]: how it starts
+    from the embedding's rows and how it ends in front of the head. A model without one passes the rows themselves."""
+
+    def open(self, rows: torch.Tensor):
+        """float32 [T, hidden] from the embedding -> what the first block's forward() gets as h."""
+        raise NotImplementedError
+
+    def close(self, h, norm: "Norm", rows: torch.Tensor) -> torch.Tensor:
+        """What the last block returned -> the final norm of the wanted rows (int32 ``rows``), in the compute dtype."""
+        raise NotImplementedError
+
+
 class Embedding(Part):
     """Token ids -> float32 rows of the residual stream."""
 
@@ -241,7 +259,7 @@ class Block:
 # ----------------------------------------------------------------------------- registries
 
 _REGISTRIES: Dict[str, Dict[str, type]] = {"mixer": {}, "feed_forward": {}, "norm": {}, "position": {}, "block": {},
-                                           "embedding": {}, "head": {}, "gate": {}}
+                                           "embedding": {}, "head": {}, "gate": {}, "connection": {}, "stream": {}}
 
 
 def _register(family: str, name: str) -> Callable[[type], type]:
@@ -261,6 +279,8 @@ def register_block(name: str): return _register("block", name)
 def register_embedding(name: str): return _register("embedding", name)
 def register_head(name: str): return _register("head", name)
 def register_gate(name: str): return _register("gate", name)
+def register_connection(name: str): return _register("connection", name)
+def register_stream(name: str): return _register("stream", name)
 
 
 def unregister(family: str, name: str) -> None:

@@ -18,7 +18,11 @@ compute dtype for the next sublayer's first matrix product.
 h <- norm_b(alpha h + feed_forward(h)), with the constant ``residual_scale`` = alpha (an option of the layer's spec);
 the feed-forward and its norm may be absent. Slots: mixer, mixer_norm, feed_forward, feed_forward_norm. The sublayers
 read h itself. Scaling, sum and norm are one float32 kernel (two mixers side by side hand over both results and their
-constants), which also leaves h in the compute dtype for the next sublayer's first matrix product."""
+constants), which also leaves h in the compute dtype for the next sublayer's first matrix product.
+
+"hyper_prenorm": prenorm over several residual streams (parts/streams.py). Slots: mixer_norm, mixer_link, mixer,
+feed_forward_norm, feed_forward_link, feed_forward (the last three may be absent together); the links are of family
+"connection". h is a ``StreamRows``; each sublayer's result stays pending there for the kernel that reads next."""
 from __future__ import annotations
 
 import os
@@ -231,4 +235,28 @@ class PostNormBlock(Block):
             norm = self.feed_forward_norm
             h, copy = ops.sum_norm(h, self.alpha, y, 1.0, None, 0.0, norm.weight, norm.eps, rt.dtype)
         step.extras["rows_copy"] = (h, copy)
+        return h
+
+
+@register_block("hyper_prenorm")
+class HyperPreNormBlock(Block):
+    def __init__(self, mixer_norm, mixer_link, mixer, feed_forward_norm=None, feed_forward_link=None, feed_forward=None):
+        parts = {"mixer_norm": mixer_norm, "mixer_link": mixer_link, "mixer": mixer}
+        if feed_forward is not None:
+            if feed_forward_norm is None or feed_forward_link is None:
+                raise ValueError("a feed-forward in a hyper_prenorm block needs its norm and its link")
+            parts.update(feed_forward_norm=feed_forward_norm, feed_forward_link=feed_forward_link, feed_forward=feed_forward)
+        super().__init__(**parts)
+        self.feed_forward = feed_forward
+        for n in (mixer_norm, feed_forward_norm):
+            if n is not None and not all(hasattr(n, a) for a in ("eps", "groups")):
+                raise ValueError("a hyper_prenorm block needs norms of the (weight, eps, groups) root-mean-square kind")
+
+    def forward(self, h, step, cache, write_cache=True):
+        dtype = self.mixer.rt.dtype
+        n = h.read(self.mixer_link, self.mixer_norm, dtype)
+        h.write(self.mixer_link, self.mixer.forward(n, step, cache, None, write_cache))
+        if self.feed_forward is not None:
+            n = h.read(self.feed_forward_link, self.feed_forward_norm, dtype)
+            h.write(self.feed_forward_link, self.feed_forward.forward(n, None))
         return h

@@ -17,6 +17,16 @@ float32 whatever the compute dtype: the six projections are one matrix product w
 
 ``names`` renames the local tensors by role (q, k, v, q_filter, k_filter, v_filter, beta, step, a_log, dt_bias, gate,
 norm, o).
+
+Kind "channel_delta_rule" is the same rule with a decay per head AND key channel, which acts on the rows of S, and with
+the decays and the output gate behind products of low rank:
+
+    g = exp(-exp(A_log[h]) * softplus(Wa2 (Wa1 x) + dt_bias))        laid out heads x dim
+    S <- diag(g) S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
+    out = Wo (o / sqrt(mean(o^2) + eps) * weight * sigmoid(Wg2 (Wg1 x)))
+
+Roles decay_low, decay_up, gate_low, gate_up take the place of step and gate. The two first factors are one product in
+the compute dtype, the two second factors one product with float32 rows (their matrices on a block diagonal).
 """
 from __future__ import annotations
 
@@ -123,6 +133,77 @@ class GatedDeltaRule(Mixer):
         o = ops.state_scan(ops.SCAN_DELTA_RULE, prep, 0, nqk, 2 * nqk, prep, self.channels, cache["S"], step.seg_start,
                            step.seg_slot, self.n_heads, self.n_heads // self.n_qk, self.dim, self.v_dim, write_cache, step.max_q_len)
         y = ops.head_norm_gate(o, self.norm_w, self.eps, rows, self.gate_col, self.n_heads, self.v_dim, self.rt.dtype)
+        if residual is None:
+            return self.o(y, out_dtype=torch.float32)
+        return self.o(y, residual=residual)
+
+
+_CHANNEL_NAMES = {"decay_low": "a_low.weight", "decay_up": "a_up.weight", "gate_low": "g_low.weight", "gate_up": "g_up.weight"}
+
+
+@register_mixer("channel_delta_rule")
+class ChannelDeltaRule(GatedDeltaRule):
+    @staticmethod
+    def _names(spec):
+        return {**_NAMES, **_CHANNEL_NAMES, **dict(spec.get("names") or {})}
+
+    @classmethod
+    def param_shapes(cls, spec):
+        H, nh, d = int(spec["hidden_size"]), int(spec["num_heads"]), int(spec["head_dim"])
+        dv = int(spec.get("v_head_dim") or d)
+        ra, rg = int(spec.get("decay_rank") or -1), int(spec.get("gate_rank") or -1)       # -1: the checkpoint's
+        n, base = cls._names(spec), _names(spec)
+        shapes = GatedDeltaRule.param_shapes(spec)
+        del shapes[base["step"]], shapes[base["gate"]]
+        shapes.update({n["dt_bias"]: (nh * d,), n["decay_low"]: (ra, H), n["decay_up"]: (nh * d, ra), n["gate_low"]: (rg, H),
+                       n["gate_up"]: (nh * dv, rg)})
+        return shapes
+
+    @classmethod
+    def init_params(cls, spec, name, shape, gen):
+        n = cls._names(spec)
+        if name in (n["decay_low"], n["decay_up"], n["gate_low"], n["gate_up"]):
+            return 0.3 * torch.randn(shape, generator=gen, dtype=torch.float32, device=gen.device)
+        return super().init_params(spec, name, shape, gen)
+
+    def load(self, params):
+        n = self._names(self.spec)
+        pad8 = lambda w, dim: torch.nn.functional.pad(w, (0, 0, 0, -w.shape[0] % 8) if dim == 0 else (0, -w.shape[1] % 8))
+        lows, ups = [], []
+        for low, up in (("decay_low", "decay_up"), ("gate_low", "gate_up")):
+            if params[n[low]].shape[0] != params[n[up]].shape[1]:
+                raise ValueError(f"the two factors of a low-rank product disagree: {tuple(params[n[low]].shape)} and {tuple(params[n[up]].shape)}")
+            lows.append(pad8(params[n[low]], 0))             # (ranks padded with zeros: rows of whole 16-byte pieces)
+            ups.append(pad8(params[n[up]], 1))
+        # result rows [q | k | v | write strengths], float32
+        self.proj = Linear(self.rt, torch.cat([params[n[r]] for r in ("q", "k", "v", "beta")], dim=0))
+        self.beta_col = self.channels
+        self.low = Linear(self.rt, torch.cat(lows, dim=0))
+        # result rows [decay logits (heads x dim) | gate logits (heads x v_dim)], float32
+        self.up = Linear(self.rt, torch.block_diag(*ups))
+        self.gate_col = self.n_heads * self.dim
+        f32 = dict(device=self.rt.device, dtype=torch.float32)
+        self.a_log = params[n["a_log"]].to(**f32).contiguous()
+        self.dt_bias = params[n["dt_bias"]].to(**f32).contiguous()
+        self.norm_w = params[n["norm"]].to(**f32).repeat(self.n_heads).contiguous()
+        self.o = Linear(self.rt, params[n["o"]])
+        if self.taps > 0:
+            self.filter_w = torch.cat([params[n["q_filter"]], params[n["k_filter"]], params[n["v_filter"]]], dim=0).to(**f32).t().contiguous()
+
+    def forward(self, x, step, cache, residual, write_cache=True):
+        rows = self.proj(x, out_dtype=torch.float32)
+        logits = self.up(self.low(x), out_dtype=torch.float32)
+        tails = cache.get("tails")
+        inline_tail = tails is not None and write_cache and step.max_q_len == 1
+        prep = ops.delta_prepare(rows, 0, 0, self.beta_col, self.filter_w, tails, self.a_log, self.dt_bias, self.unit_eps,
+                                 float(self.dim) ** -0.5, step, self.n_heads, self.n_qk, self.dim, self.v_dim, inline_tail, logits, 0)
+        if tails is not None and write_cache and not inline_tail:
+            ops.tail_update(rows, 0, tails, step.seg_start, step.seg_slot)
+        nqk = self.n_qk * self.dim
+        decay_col, scalar_col = ops.delta_columns(self.n_heads, self.n_qk, self.dim, self.v_dim, True)
+        o = ops.state_scan(ops.SCAN_CHANNEL_DELTA, prep, 0, nqk, 2 * nqk, prep, decay_col, cache["S"], step.seg_start, step.seg_slot,
+                           self.n_heads, self.n_heads // self.n_qk, self.dim, self.v_dim, write_cache, step.max_q_len, scalar_col=scalar_col)
+        y = ops.group_norm_gate(o, self.norm_w, self.eps, logits, self.gate_col, "sigmoid", self.n_heads, self.v_dim, self.rt.dtype)
         if residual is None:
             return self.o(y, out_dtype=torch.float32)
         return self.o(y, residual=residual)

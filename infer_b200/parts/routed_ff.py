@@ -24,7 +24,9 @@ Other forms, each a key of the spec:
                  s + correction are chosen (``correction`` [experts], a stored tensor that only the choice sees);
                  weight_e = s_e as it is, not renormalised; no groups. "softmax_top": the ``top`` experts with the
                  largest logits are chosen and their weights are the softmax over the chosen logits only (which is
-                 what the form above gives without groups and with sum_eps 0); no groups
+                 what the form above gives without groups and with sum_eps 0); no groups. "sigmoid_groups":
+                 s = sigmoid(x Wr^T); groups as above, a group's score being the sum of its two largest s;
+                 weight_e = s_e as it is, not renormalised
 ``expert_kind``  "clipped_swish_glu" (above), "relu_squared": expert(x) = Wd relu(Wu x)^2, no gate matrix, no limit, or
                  "swish_glu": expert(x) = Wd (g sigmoid(g) * u) with g = Wg x, u = Wu x, no limit
 ``out_scale``    a constant on the result (default 1), multiplied into the experts' weights in float32: a block's
@@ -57,12 +59,12 @@ class RoutedExperts(FeedForward):
             if self.groups != 1 or self.keep != 1:
                 raise ValueError("a softmax_top router has no groups")
             self.sum_eps = 0.0
-        if self.router_kind not in ("softmax_groups", "sigmoid", "softmax_top") or \
+        if self.router_kind not in ("softmax_groups", "sigmoid", "softmax_top", "sigmoid_groups") or \
                 self.expert_kind not in ("clipped_swish_glu", "relu_squared", "swish_glu"):
             raise ValueError(f"routed_experts: unknown router_kind {self.router_kind!r} or expert_kind {self.expert_kind!r}")
         if self.router_kind == "sigmoid" and (self.groups != 1 or self.keep != 1):
             raise ValueError("a sigmoid router has no groups")
-        if self.out_scale != 1.0 and (self.router_kind != "sigmoid" or self.shared_ff):
+        if self.out_scale != 1.0 and (self.router_kind not in ("sigmoid", "sigmoid_groups") or self.shared_ff):
             raise ValueError("out_scale goes into the weights of a sigmoid router and does not reach a shared expert")
         self.correction = None
         if min(self.hidden, self.n_experts, self.top, self.groups, self.keep, self.ff) <= 0 or self.shared_ff < 0:
@@ -113,6 +115,8 @@ class RoutedExperts(FeedForward):
         logits = self.router(x, out_dtype=torch.float32)
         if self.router_kind == "sigmoid":
             weights, _ = ops.route_sigmoid(logits, self.correction, self.top, self.out_scale)
+        elif self.router_kind == "sigmoid_groups":
+            weights, _ = ops.route(logits, self.top, self.groups, self.keep, sigmoid=True, group_best=2, renormalise=False, mult=self.out_scale)
         else:
             weights, _ = ops.route(logits, self.top, self.groups, self.keep, self.sum_eps)
         rows = self.gate_up(x)

@@ -8,6 +8,8 @@ registers its own ``Embedding`` / ``Head`` kinds; the model only calls ``forward
 renames the part's one tensor (default "weight") under its prefix. A head with ``logit_scale`` and / or ``softcap``
 returns cap * tanh(logits * scale / cap) (the scale alone without a cap). With ``norm_weight_name`` (and ``norm_eps``) the
 looked-up rows are divided by their root mean square and multiplied by that weight before they enter the residual stream.
+With ``sinusoid_base`` = b a position vector is added to the (scaled) rows: channels 2i and 2i + 1 take sin and cos of
+position * b^(-2i / hidden); the angles are formed in float64 and brought into one turn before the float32 functions.
 """
 from __future__ import annotations
 
@@ -34,6 +36,10 @@ class TokenTable(Embedding):
         if self.norm_name is not None and self.norm_eps <= 0:
             raise ValueError("a norm behind the token table needs a positive norm_eps")
         self.norm_weight = None
+        self.sinusoid_base = spec.get("sinusoid_base")
+        if self.sinusoid_base is not None and (float(self.sinusoid_base) <= 0 or self.norm_name is not None):
+            raise ValueError("sinusoidal positions need a positive base and do not combine with a norm behind the table")
+        self.freq = None
 
     @classmethod
     def param_shapes(cls, spec):
@@ -51,6 +57,9 @@ class TokenTable(Embedding):
     def load(self, params):
         # The table is read row by row; it keeps the compute dtype of the matrices (a tied head multiplies by it).
         self.weight = params[str(self.spec.get("weight_name", "weight"))].to(device=self.rt.device, dtype=self.rt.dtype).contiguous()
+        if self.sinusoid_base is not None:
+            i = torch.arange((self.hidden + 1) // 2, dtype=torch.float64)
+            self.freq = torch.pow(torch.tensor(float(self.sinusoid_base), dtype=torch.float64), -2.0 * i / self.hidden).to(self.rt.device).contiguous()
         if self.norm_name is not None:
             self.norm_weight = params[str(self.norm_name)].to(device=self.rt.device, dtype=torch.float32).contiguous()
 
@@ -58,6 +67,9 @@ class TokenTable(Embedding):
         return self.weight
 
     def forward(self, step):
+        if self.freq is not None:
+            return ops.embedding_sinusoid(self.weight, step.token_ids, step.positions, self.freq, step.status,
+                                          getattr(step, "feedback", None), step.token_seg, step.seg_slot, self.scale)
         rows = ops.embedding(self.weight, step.token_ids, step.status, getattr(step, "feedback", None),
                              step.token_seg, step.seg_slot, self.scale)
         if self.norm_weight is not None:
