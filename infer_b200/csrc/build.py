@@ -35,6 +35,7 @@ MODULES: Dict[str, str] = {
     "post": "post_ops.cu",       # norms after the residual sum, per-head query/key norms, mixtures with the token before
     "stream": "stream_ops.cu",   # several residual streams, norms over groups of channels, sinusoidal positions
     "talk": "talk_ops.cu",       # attention whose heads exchange their scores before the softmax
+    "talk_pf": "talk_prefill.cu",       # the same attention for prompt portions on the tensor cores
     "latent_pf": "latent_prefill.cu",   # the same attention for prompt portions: per-head keys and values, tensor cores
     "gemvb": "gemv_bulk.cu",
     "gemm": "gemm_tcgen05.cu",
@@ -42,9 +43,10 @@ MODULES: Dict[str, str] = {
     "attn_tc": "attention_tc.cu",
     "capi": "capi.cpp",          # host code only: the C handle API over the engine (needs the interpreter's headers)
 }
-HEADERS = ["common.cuh", "gemm_static.h", "tma_map.cuh"]
+HEADERS = ["common.cuh", "gemm_static.h", "tc_ops.cuh", "tma_map.cuh"]
 # modules that are compiled per model size: the variant that build_all() makes (others are built at first use)
-DEFAULT_DEFINES = {"attn": {"IB_HEAD_DIM": 128}, "attn_tc": {"IB_HEAD_DIM": 128}, "latent_pf": {"IB_QK_DIM": 128, "IB_V_DIM": 128}}
+DEFAULT_DEFINES = {"attn": {"IB_HEAD_DIM": 128}, "attn_tc": {"IB_HEAD_DIM": 128}, "latent_pf": {"IB_QK_DIM": 128, "IB_V_DIM": 128},
+                   "talk_pf": {"IB_HEAD_DIM": 128, "IB_V_DIM": 128, "IB_HEADS": 12}}
 
 
 class BuildError(RuntimeError):

@@ -375,6 +375,58 @@ def attention_prefill_biased(q, k_cache, v_cache, block_table, step, n_heads, n_
     return out
 
 
+# Attention whose heads exchange their scores (talk_prefill.cu): sizes that the tensor-core kernels are built for, and how
+# much memory a launch's scores may take (a launch covers as many query tiles of 128 tokens as fit).
+TALK_PREFILL_DIMS, TALK_PREFILL_MAX_HEADS = (64, 128), 32
+TALK_SCORES_MAX_BYTES = 512 << 20
+
+
+def talk_key_tiles(max_ctx_len: int, window: Optional[int], chunk: Optional[int]) -> int:
+    """The most key tiles of 128 (aligned to absolute positions) that 128 neighbouring queries see."""
+    n = -(-max_ctx_len // 128)
+    seen = min([int(v) for v in (window, chunk) if v], default=None)
+    if seen is not None:
+        n = min(n, (seen + 127 + 126) // 128 + 1)
+    return max(1, n)
+
+
+def talk_attention_prefill(q: torch.Tensor, q_col: int, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor, step,
+                           n_heads: int, n_kv: int, head_dim: int, v_head_dim: int, window: Optional[int], chunk: Optional[int],
+                           scale: float, cap: float, talk: Optional[torch.Tensor]) -> Optional[torch.Tensor]:
+    """``ops.talk_attention`` of the step's segments of two or more tokens on the tensor cores; the rows of one-token
+    segments are left unwritten. None if the shape is refused. The library is compiled for these sizes at first use."""
+    if not ATTENTION_TC or head_dim not in TALK_PREFILL_DIMS or v_head_dim not in TALK_PREFILL_DIMS or n_heads > TALK_PREFILL_MAX_HEADS:
+        return None
+    T, ld, n_pages, page_size = ops._check_talk(q, q_col, k_cache, v_cache, block_table, n_heads, n_kv, head_dim, v_head_dim, talk)
+    if q.dtype != torch.bfloat16 or q_col % 8 or ld % 8 or page_size != 16:
+        return None
+    defines = {"IB_HEAD_DIM": head_dim, "IB_V_DIM": v_head_dim, "IB_HEADS": n_heads}
+    if not _fn("talk_pf", "ib_talk_prefill_fits", [c_int] * 5, defines)(n_heads, n_kv, head_dim, v_head_dim, page_size):
+        return None
+    st = device_state(q.device)
+    n_long = sum(1 for n in step.seg_lens if n > 1)
+    tiles = talk_key_tiles(step.max_ctx_len, window, chunk)
+    n_qt = -(-step.max_q_len // 128)
+    per_qt = n_long * n_heads * tiles * 128 * 128
+    at_once = max(1, min(n_qt, TALK_SCORES_MAX_BYTES // (4 * per_qt)))
+    scores = torch.empty(per_qt * at_once, dtype=torch.float32, device=q.device)
+    out = torch.empty((T, n_heads * v_head_dim), dtype=q.dtype, device=q.device)
+    f = _fn("talk_pf", "ib_talk_prefill", [c_void_p, c_int64, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int,
+                                           c_int64] + [c_int] * 7 + [c_float, c_float, c_void_p, c_int64] + [c_int] * 4 +
+            [c_void_p, c_int64, c_int, c_void_p, c_void_p], defines)
+    for qt0 in range(0, n_qt, at_once):
+        n = min(at_once, n_qt - qt0)
+        # few (query tile, key tile) pairs: several CTAs share one (about half of the pairs of a causal prompt exist)
+        pairs, q_split = n_long * n * tiles, 1
+        while q_split < 4 and pairs * q_split < 2 * st.sm_count:
+            q_split *= 2
+        _call(f, q.data_ptr(), ld, int(q_col), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), block_table.data_ptr(),
+              block_table.shape[1], step.seg_start.data_ptr(), step.seg_pos0.data_ptr(), step.seg_pos0.numel(), T, n_heads, n_kv, head_dim,
+              v_head_dim, page_size, int(window or 0), int(chunk or 0), float(scale), float(cap or 0.0), _ptr(talk), n_pages, qt0, n, tiles,
+              q_split, scores.data_ptr(), scores.numel(), n_long, st.status.data_ptr(), _stream())
+    return out
+
+
 def decode_fused_supported(n_heads: int, n_kv: int, head_dim: int, page_size: int) -> bool:
     return attention_supported(n_heads, n_kv, head_dim, page_size) and head_dim % 32 == 0
 

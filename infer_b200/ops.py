@@ -1417,3 +1417,38 @@ def talk_attention(q: torch.Tensor, q_col: int, k_cache: torch.Tensor, v_cache: 
           v_head_dim, page_size, int(window or 0), int(chunk or 0), float(scale), float(cap or 0.0), _ptr(talk), n_pages,
           dtype_code(q.dtype), _ptr(step.status), _stream())
     return out
+
+
+def talk_split_fits(n_heads: int, n_kv: int, head_dim: int, v_head_dim: int, page_size: int) -> bool:
+    return bool(_fn("talk", "ib_talk_split_fits", [c_int] * 5)(int(n_heads), int(n_kv), int(head_dim), int(v_head_dim), int(page_size)))
+
+
+def talk_attention_split(q: torch.Tensor, q_col: int, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor, step,
+                         n_heads: int, n_kv: int, head_dim: int, v_head_dim: int, window: Optional[int], chunk: Optional[int], scale: float,
+                         cap: float, talk: Optional[torch.Tensor], out: Optional[torch.Tensor] = None, single_only: bool = False,
+                         fresh_cols=None) -> Optional[torch.Tensor]:
+    """``talk_attention`` of single tokens in bfloat16 with their keys split over CTAs (chunks of 64 keys aligned to
+    absolute positions); None where the sizes are refused. With ``single_only`` only tokens that are a segment of their
+    own are computed, into ``out``. ``fresh_cols`` (first column of the keys, of the values; only for steps of one token per
+    request): the tokens' own keys and values are still in the rows q and are stored to their pages here."""
+    T, ld, n_pages, page_size = _check_talk(q, q_col, k_cache, v_cache, block_table, n_heads, n_kv, head_dim, v_head_dim, talk)
+    if q.dtype != torch.bfloat16 or q_col % 8 or ld % 8 or not talk_split_fits(n_heads, n_kv, head_dim, v_head_dim, page_size):
+        return None
+    if fresh_cols is not None and (fresh_cols[0] % 8 or fresh_cols[1] % 8 or fresh_cols[0] + n_kv * head_dim > ld or fresh_cols[1] + n_kv * v_head_dim > ld):
+        return None
+    if out is None:
+        out = torch.empty((T, n_heads * v_head_dim), dtype=q.dtype, device=q.device)
+    else:
+        _check(out, "out", q.dtype, (T, n_heads * v_head_dim))
+    visible = min([int(step.max_ctx_len)] + [int(v) for v in (window, chunk) if v])
+    n_chunks = int(_fn("talk", "ib_talk_split_chunks", [c_int])(max(visible, 1)))
+    ws = torch.empty(T * n_heads * n_chunks * (v_head_dim + 2), dtype=torch.float32, device=q.device)
+    f = _fn("talk", "ib_talk_attention_split", [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int64] +
+            [c_void_p] * 5 + [c_int64] + [c_int] * 8 + [c_float, c_float, c_void_p, c_int64, c_void_p, c_void_p])
+    _call(f, q.data_ptr() + q_col * q.element_size(), ld, q.data_ptr() if fresh_cols is not None else None, ld,
+          int(fresh_cols[0]) if fresh_cols else 0, int(fresh_cols[1]) if fresh_cols else 0, k_cache.data_ptr(), v_cache.data_ptr(),
+          block_table.data_ptr(), block_table.shape[1], step.token_seg.data_ptr(), step.positions.data_ptr(),
+          step.seg_start.data_ptr() if single_only else None, out.data_ptr(), ws.data_ptr(), T, n_heads, n_kv, head_dim, v_head_dim,
+          page_size, int(window or 0), int(chunk or 0), n_chunks, float(scale), float(cap or 0.0), _ptr(talk), n_pages, _ptr(step.status),
+          _stream())
+    return out

@@ -372,11 +372,27 @@ class Attention(Mixer):
         """Capped scores, the exchange among the heads and chunks. The part's columns [q | k | v] start at ``col0``; keys
         and values go to the pages as projected, the attention kernels read the queries where they are."""
         table = step.block_tables[cache.group]
-        nq, nk = self.n_heads * self.head_dim, self.n_kv * self.head_dim
+        k_col = col0 + self.n_heads * self.head_dim
+        v_col = k_col + self.n_kv * self.head_dim
+        args = (qkv, col0, cache.k, cache.v, table, step, self.n_heads, self.n_kv, self.head_dim, self.v_dim, self.window, self.chunk,
+                self.scale, self.cap, self.talk_w)
+        fast = self.rt.fast("attention")
+        if fast and step.max_q_len <= 1:
+            # single tokens: the kernel that splits a token's keys over CTAs also stores the token's own key and value
+            ctx = ops.talk_attention_split(*args, fresh_cols=(k_col, v_col) if write_cache else None)
+            if ctx is not None:
+                return self._project_out(ctx, residual)
         if write_cache:
-            ops.kv_store(qkv, col0 + nq, col0 + nq + nk, step, table, cache.k, cache.v, self.n_kv, self.head_dim, self.v_dim)
-        ctx = ops.talk_attention(qkv, col0, cache.k, cache.v, table, step, self.n_heads, self.n_kv, self.head_dim, self.v_dim, self.window,
-                                 self.chunk, self.scale, self.cap, self.talk_w)
+            ops.kv_store(qkv, k_col, v_col, step, table, cache.k, cache.v, self.n_kv, self.head_dim, self.v_dim)
+        ctx = None
+        if fast and step.max_q_len > 1:
+            from .. import fast_ops
+            ctx = fast_ops.talk_attention_prefill(*args)
+            if ctx is not None and any(n == 1 for n in step.seg_lens):
+                # one-token segments beside prompt portions, into the same rows
+                ctx = ops.talk_attention_split(*args, out=ctx, single_only=True)
+        if ctx is None:
+            ctx = ops.talk_attention(*args)
         return self._project_out(ctx, residual)
 
     def forward(self, x, step, cache, residual, write_cache=True):
