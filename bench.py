@@ -6,6 +6,7 @@ random weights on one B200.
     python bench.py --design fozerax [--sizes 1.5b|7b] [--layers L]     (beside Ruvenex, the closest design, and Qwen2)
     python bench.py --design pefazen [--sizes 1.5b|7b] [--layers L]     (beside Fozerax, the closest design, and Qwen2)
     python bench.py --design biravik [--sizes 1.5b|7b] [--layers L]     (beside Fozerax, the closest design, and Qwen2)
+    python bench.py --design notirax [--sizes 1.5b|7b] [--layers L]     (beside Fozerax, the closest design, and Qwen2)
 
 Prints ONE JSON line. "value" is decoded tokens per second of the step function, timed on the device with CUDA
 events around K decode steps of a batch of 8 requests whose 2,048-token contexts already lie in the paged cache
@@ -37,9 +38,10 @@ def _preset(name):
 SIZES = {"1.5b": _preset("qwen2.5-1.5b"), "7b": _preset("qwen2.5-7b"), "14b": _preset("qwen2.5-14b")}
 # Other designs at the same layer sizes (width, heads, feed-forward), for --design.
 DESIGNS = {"ruvenex": {"1.5b": "ruvenex-1.5b", "7b": "ruvenex-7b"}, "fozerax": {"1.5b": "fozerax-1.5b", "7b": "fozerax-7b"},
-           "pefazen": {"1.5b": "pefazen-1.5b", "7b": "pefazen-7b"}, "biravik": {"1.5b": "biravik-1.5b", "7b": "biravik-7b"}}
+           "pefazen": {"1.5b": "pefazen-1.5b", "7b": "pefazen-7b"}, "biravik": {"1.5b": "biravik-1.5b", "7b": "biravik-7b"},
+           "notirax": {"1.5b": "notirax-1.5b", "7b": "notirax-7b"}}
 # the designs a design is measured beside, besides Qwen2: the closest one the engine has
-BESIDE = {"fozerax": ["ruvenex"], "pefazen": ["fozerax"], "biravik": ["fozerax"]}
+BESIDE = {"fozerax": ["ruvenex"], "pefazen": ["fozerax"], "biravik": ["fozerax"], "notirax": ["fozerax"]}
 CONFIG = SIZES["1.5b"]
 FALLBACK_PEAKS = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "bf16_tflops_sustained": 1400.0}
 
@@ -164,7 +166,11 @@ def decode_bytes(eng, batch, context_mid):
     head_w = getattr(getattr(eng.model.head, "linear", None), "weight", None)
     if table is not None and (head_w is None or head_w.data_ptr() != table.data_ptr()):
         w -= table.numel() * item - batch * spec.hidden_size * item         # an untied table is read row by row only
-    kv = sum(len(g.cache_ids) * g.need.num_kv_heads * (g.need.head_dim + g.need.value_dim) * item for g in eng.cache.groups)
+    def positions(need):                   # that a token at position context_mid reads
+        n = context_mid if need.window is None else min(context_mid, need.window + min(need.keep_first, max(0, context_mid - need.window)))
+        return n if need.chunk is None else min(n, context_mid % need.chunk + 1)
+    kv = sum(len(g.cache_ids) * g.need.num_kv_heads * (g.need.head_dim + g.need.value_dim) * item * positions(g.need)
+             for g in eng.cache.groups) / max(context_mid, 1)
     state = sum(t[0].numel() * t.element_size() for tensors in eng.cache.state.values() for t in tensors.values())
     return w + batch * (context_mid * kv + 2 * state), w, kv          # a request's fixed-size state is read and written
 
@@ -447,6 +453,28 @@ def biravik_flops(cfg, T):
     return total + 2 * W * cfg["vocab"]
 
 
+def notirax_flops(cfg, T):
+    """Arithmetic of a prompt of T tokens through a Notirax configuration as the design states it: the projections,
+    attention scores, their exchange among the heads and the sums over what a query sees, the recurrence's state updates
+    and read-outs, and the chosen experts only."""
+    W, total = cfg["width"], 0.0
+    for l in cfg["layers"]:
+        m = l["mixer"]
+        H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        if l["type"] == "attention":
+            total += 2 * T * W * ((H + G) * d + (G + H) * dv)
+            c = min(T, (m.get("mask") or {}).get("size") or T)
+            seen = T // c * (c * (c + 1) / 2) + (T % c) * (T % c + 1) / 2
+            total += 2 * H * (d + dv + H) * seen
+        else:
+            ra, rg = m.get("decay_rank", d), m.get("gate_rank", d)
+            total += 2 * T * W * (2 * G * d + 2 * H * dv + H + ra + rg) + 2 * T * H * (d * ra + dv * rg) + T * H * d * dv * 9
+        f = l["mlp"]
+        if f:
+            total += 2 * T * W * (3 * f["router"]["top"] * f["expert"]["ff"] + f["router"]["experts"])
+    return total + 2 * W * cfg["vocab"]
+
+
 def design_flops(cfg, T):
     """Arithmetic of a prompt of T tokens through a model of --design's configuration (matrix products, attention
     scores and sums, the recurrence's state updates and read-outs), logits at the last place only."""
@@ -456,6 +484,8 @@ def design_flops(cfg, T):
         return pefazen_flops(cfg, T)
     if cfg.get("architecture") == "Biravik":
         return biravik_flops(cfg, T)
+    if cfg.get("architecture") == "Notirax":
+        return notirax_flops(cfg, T)
     W, total = cfg["width"], 0.0
     for l in cfg["layers"]:
         a, r = l["mixer"]["left"], l["mixer"]["right"]
