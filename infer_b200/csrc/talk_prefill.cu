@@ -11,8 +11,9 @@
 // positions, all heads, are the columns: 16 columns of tensor memory per head, all heads side by side, so that the
 // thread that owns a key reads every head's score of its (query, key) pairs with no exchange between threads:
 //   warp 0      TMA producer: the key tile, then the queries through a ring (a kv head's group of heads per stage)
-//   warp 1      MMA issuer: 16 columns per head, the blocks of 16 queries in two tensor-memory buffers where they fit
-//   warps 2..9  thread = (key, half of the block's queries): scale and cap, then score_h = sum_g talk[h, g] score_g for four
+//   warp 1      MMA issuer: the heads of a kv head in one product (a product of few columns costs the tensor core
+//               as much as one of a hundred), the blocks of 16 queries in two tensor-memory buffers where they fit
+//   the others  thread = (key, share of the block's queries): scale and cap, then score_h = sum_g talk[h, g] score_g for four
 //               queries at a time in packed float pairs, and a 16-byte store per head (a warp: 512 bytes)
 // Kernel 2 (softmax and values): one CTA per (query tile, head), the softmax and P V of the engine's prompt attention
 // (attention_tc.cu) with the scores copied in by bulk copies instead of computed. It masks; kernel 1 writes whatever
@@ -135,16 +136,18 @@ __device__ __forceinline__ int page_at(const Params& p, int seg, int key) {
 // ------------------------------------------------------------------------------------------------ kernel 1
 constexpr int NQ = 16;                       // queries of a block
 constexpr int BLOCKS = BM / NQ;
-constexpr int MIX_WARPS = 8;
+constexpr int MIX_WARPS = H <= 16 ? 16 : 8;   // (by the registers that H scores of four queries take)
+constexpr int Q_SHARES = MIX_WARPS / 4;      // warps that own the same keys share a block's queries
+constexpr int PASSES = NQ / 4 / Q_SHARES;    // of four queries each
 constexpr int SCORE_THREADS = 64 + MIX_WARPS * 32;
 constexpr int S_BUFS = 2 * H * NQ <= 512 ? 2 : 1;
 constexpr int s_cols(int need) { return need <= 32 ? 32 : (need <= 64 ? 64 : (need <= 128 ? 128 : (need <= 256 ? 256 : 512))); }
 constexpr int S_TMEM = s_cols(S_BUFS * H * NQ);
-constexpr int HP = (H + 1) & ~1;             // heads rounded up to an even count
+constexpr int HP = (H + 3) & ~3;             // heads rounded up to a multiple of four
 constexpr int MAX_STAGES = 4;
 constexpr int K_HEAD_BYTES = DB * BN * 128;  // one kv head's key tile
 constexpr int Q_HEAD_BYTES = DB * NQ * 128;  // one head's queries of a block
-constexpr int SCORE_FIXED = H * HP * 8 + 1024 + 256;
+constexpr int SCORE_FIXED = H * HP * 4 + 1024 + 256;
 
 __global__ void __launch_bounds__(SCORE_THREADS)
 talk_scores_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k, const Params p) {
@@ -154,9 +157,9 @@ talk_scores_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
     const int group = H / p.n_kv, stage_bytes = group * Q_HEAD_BYTES;
     const uint32_t k_s = base, q_s = k_s + p.n_kv * K_HEAD_BYTES;
     uint8_t* tail = base_ptr + p.n_kv * K_HEAD_BYTES + p.n_stages * stage_bytes;
-    uint64_t* T2 = reinterpret_cast<uint64_t*>(tail);        // [H][HP] the exchange matrix, every entry twice
-    const uint32_t bars = base + uint32_t(tail - base_ptr) + H * HP * 8;
-    volatile uint32_t* slots = reinterpret_cast<volatile uint32_t*>(tail + H * HP * 8 + 128);    // [0] TMEM base, [1] abort
+    float* T_s = reinterpret_cast<float*>(tail);             // [H][HP] the exchange matrix
+    const uint32_t bars = base + uint32_t(tail - base_ptr) + H * HP * 4;
+    volatile uint32_t* slots = reinterpret_cast<volatile uint32_t*>(tail + H * HP * 4 + 128);    // [0] TMEM base, [1] abort
     const uint32_t k_full = bars, q_full = bars + 8, q_empty = q_full + 8 * MAX_STAGES, s_full = q_empty + 8 * MAX_STAGES,
                    s_empty = s_full + 16;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -180,8 +183,7 @@ talk_scores_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
     if (p.talk) {
         for (int i = threadIdx.x; i < H * HP; i += SCORE_THREADS) {
             const int h = i / HP, g = i - h * HP;
-            const float v = g < H ? p.talk[h * H + g] : 0.0f;
-            T2[i] = pack2(v, v);
+            T_s[i] = g < H ? p.talk[h * H + g] : 0.0f;
         }
     }
     if (threadIdx.x == 0) {
@@ -235,7 +237,7 @@ talk_scores_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
                 __syncwarp();
                 for (int i = lane; i < group * DB; i += 32) {
                     const int hq = i / DB, db = i - hq * DB;
-                    tma_load_2d(q_s + st * stage_bytes + hq * Q_HEAD_BYTES + db * (NQ * 128), &tm_q, q_full + 8 * st,
+                    tma_load_2d(q_s + st * stage_bytes + (db * group + hq) * (NQ * 128), &tm_q, q_full + 8 * st,
                                 p.q_col + (g * group + hq) * D + db * 64, w.t0 + qt * BM + b * NQ);
                 }
             }
@@ -249,7 +251,7 @@ talk_scores_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
     } else if (warp == 1) {
         // ---------------------------------------------------------------- MMA issuer
         if (lane == 0) {
-            constexpr uint32_t idesc = make_idesc(NQ, false);
+            const uint32_t idesc = make_idesc(group * NQ, false);
             bool ok = mbar_wait(k_full, 0);
             tc_fence_after();
             int n = 0, nb = 0;
@@ -262,16 +264,15 @@ talk_scores_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
                     ok = mbar_wait(q_full + 8 * st, (n / p.n_stages) & 1);
                     if (!ok) break;
                     tc_fence_after();
-                    for (int hq = 0; hq < group; hq++) {
-                        const uint32_t dst = tmem_base + buf * (H * NQ) + (g * group + hq) * NQ;
+                    // one product per 16 channels for all heads of the group: 16 * group columns
+                    const uint32_t dst = tmem_base + buf * (H * NQ) + g * group * NQ;
 #pragma unroll
-                        for (int db = 0; db < DB; db++) {
-                            const uint64_t kd = make_desc(k_s + g * K_HEAD_BYTES + db * (BN * 128), 16, 1024);
-                            const uint64_t qd = make_desc(q_s + st * stage_bytes + hq * Q_HEAD_BYTES + db * (NQ * 128), 16, 1024);
+                    for (int db = 0; db < DB; db++) {
+                        const uint64_t kd = make_desc(k_s + g * K_HEAD_BYTES + db * (BN * 128), 16, 1024);
+                        const uint64_t qd = make_desc(q_s + st * stage_bytes + db * group * (NQ * 128), 16, 1024);
 #pragma unroll
-                            for (int k = 0; k < 4; k++)      // 16 elements of the head per step = 32 bytes = 2 address units
-                                umma_f16(dst, kd + uint64_t(2 * k), qd + uint64_t(2 * k), idesc, (db > 0 || k > 0) ? 1u : 0u);
-                        }
+                        for (int k = 0; k < 4; k++)          // 16 elements of the head per step = 32 bytes = 2 address units
+                            umma_f16(dst, kd + uint64_t(2 * k), qd + uint64_t(2 * k), idesc, (db > 0 || k > 0) ? 1u : 0u);
                     }
                     umma_commit(q_empty + 8 * st);
                 }
@@ -280,8 +281,8 @@ talk_scores_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
             if (!ok) { if (!slots[1]) atomicExch(p.status, STATUS_TIMEOUT); slots[1] = 1; }
         }
     } else {
-        // ---------------------------------------------------------------- cap, exchange, store (warps 2..9)
-        const int quad = warp & 3, half = (warp - 2) >> 2;
+        // ---------------------------------------------------------------- cap, exchange, store (warps 2 and on)
+        const int quad = warp & 3, q_share = (warp - 2) >> 2;
         const int key = quad * 32 + lane;                    // key of the tile = TMEM lane
         const uint32_t lane_addr = tmem_base + (uint32_t(quad * 32) << 16);
         const float two_y = p.cap > 0.0f ? 2.0f * LOG2E * p.scale / p.cap : 0.0f, cap = p.cap, scale = p.scale;
@@ -296,16 +297,17 @@ talk_scores_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
             if (!ok) break;
             tc_fence_after();
 #pragma unroll 1
-            for (int pass = 0; pass < NQ / 8; pass++) {
-                const int i0 = half * (NQ / 2) + pass * 4;   // four queries of the block
-                uint64_t s01[HP], s23[HP];
+            for (int pass = 0; pass < PASSES; pass++) {
+                const int i0 = (q_share * PASSES + pass) * 4;   // four queries of the block
+                uint64_t s2[HP / 2][4];                      // the scores of two neighbouring heads, per query
                 {
                     float s[HP][4];
 #pragma unroll
                     for (int g = 0; g < H; g++) tmem_ld4(lane_addr + buf * (H * NQ) + g * NQ + i0, s[g]);
                     tmem_ld_wait();
-                    if (H < HP) s[HP - 1][0] = s[HP - 1][1] = s[HP - 1][2] = s[HP - 1][3] = 0.0f;
-                    if (pass == NQ / 8 - 1) {                // everything this thread reads of the buffer has arrived
+#pragma unroll
+                    for (int g = H; g < HP; g++) s[g][0] = s[g][1] = s[g][2] = s[g][3] = 0.0f;
+                    if (pass == PASSES - 1) {                // everything this thread reads of the buffer has arrived
                         tc_fence_before();
                         __syncwarp();
                         if (lane == 0) mbar_arrive(s_empty + 8 * buf);
@@ -320,33 +322,41 @@ talk_scores_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
                         }
                     }
 #pragma unroll
-                    for (int g = 0; g < HP; g++) {
-                        s01[g] = pack2(s[g][0], s[g][1]);
-                        s23[g] = pack2(s[g][2], s[g][3]);
-                    }
+                    for (int g = 0; g < HP / 2; g++)
+#pragma unroll
+                        for (int e = 0; e < 4; e++) s2[g][e] = pack2(s[2 * g][e], s[2 * g + 1][e]);
                 }
                 float* dst = dst0 + (b * NQ + i0) / 4 * (4 * BN);
                 if (p.talk) {
-#pragma unroll 1
+#pragma unroll 2
                     for (int h = 0; h < H; h++) {
-                        uint64_t a01 = 0, a23 = 0, c01 = 0, c23 = 0;     // (two chains: even and odd heads)
-                        const ulonglong2* row = reinterpret_cast<const ulonglong2*>(T2 + h * HP);
+                        // even and odd heads are summed in the two halves of a pair
+                        uint64_t acc[4] = {0, 0, 0, 0};
+                        const ulonglong2* row = reinterpret_cast<const ulonglong2*>(T_s + h * HP);
 #pragma unroll
-                        for (int g = 0; g < HP / 2; g++) {
+                        for (int g = 0; g < HP / 4; g++) {
                             const ulonglong2 t = row[g];
-                            a01 = fma2(t.x, s01[2 * g], a01);
-                            a23 = fma2(t.x, s23[2 * g], a23);
-                            c01 = fma2(t.y, s01[2 * g + 1], c01);
-                            c23 = fma2(t.y, s23[2 * g + 1], c23);
+#pragma unroll
+                            for (int e = 0; e < 4; e++) acc[e] = fma2(t.y, s2[2 * g + 1][e], fma2(t.x, s2[2 * g][e], acc[e]));
                         }
-                        const float2 x = unpack2(a01), y = unpack2(a23), u = unpack2(c01), v = unpack2(c23);
-                        *reinterpret_cast<float4*>(dst + h * head_stride) = make_float4(x.x + u.x, x.y + u.y, y.x + v.x, y.y + v.y);
+                        float o[4];
+#pragma unroll
+                        for (int e = 0; e < 4; e++) {
+                            const float2 x = unpack2(acc[e]);
+                            o[e] = x.x + x.y;
+                        }
+                        *reinterpret_cast<float4*>(dst + h * head_stride) = make_float4(o[0], o[1], o[2], o[3]);
                     }
                 } else {
 #pragma unroll
                     for (int h = 0; h < H; h++) {
-                        const float2 x = unpack2(s01[h]), y = unpack2(s23[h]);
-                        *reinterpret_cast<float4*>(dst + h * head_stride) = make_float4(x.x, x.y, y.x, y.y);
+                        float o[4];
+#pragma unroll
+                        for (int e = 0; e < 4; e++) {
+                            const float2 x = unpack2(s2[h / 2][e]);
+                            o[e] = h & 1 ? x.y : x.x;
+                        }
+                        *reinterpret_cast<float4*>(dst + h * head_stride) = make_float4(o[0], o[1], o[2], o[3]);
                     }
                 }
             }
@@ -612,7 +622,7 @@ IB_EXPORT int64_t ib_talk_prefill_tile_floats() { return TILE_FLOATS; }
 
 // 1 if this build takes these sizes.
 IB_EXPORT int ib_talk_prefill_fits(int n_heads, int n_kv, int d, int dv, int page_size) {
-    return n_heads == H && d == D && dv == DV && page_size == PAGE && n_kv > 0 && H % n_kv == 0 && ring_stages(n_kv) > 0;
+    return n_heads == H && d == D && dv == DV && page_size == PAGE && n_kv > 0 && H % n_kv == 0 && H / n_kv <= 16 && ring_stages(n_kv) > 0;
 }
 
 // Attention of the segments with two or more tokens (others are skipped), their query tiles qt0 .. qt0 + n_qt - 1 of 128

@@ -390,6 +390,21 @@ def talk_key_tiles(max_ctx_len: int, window: Optional[int], chunk: Optional[int]
     return max(1, n)
 
 
+TALK_START_BLOCKS = 2             # what starting a CTA of the score kernel costs, in blocks of 16 queries (of eight a query tile has)
+
+
+def talk_q_split(sm_count: int, lens, max_ctx_len: int, window: Optional[int], chunk: Optional[int], qt0: int, n_qt: int) -> int:
+    """How many CTAs share a (query tile, key tile) pair of the score kernel: rounds over the SMs times the time of a CTA.
+    Counts the pairs of portions that end at max_ctx_len (captured steps know no more); any answer is correct."""
+    pairs = 0
+    for m in lens:
+        for qt in range(qt0, min(qt0 + n_qt, -(-m // 128))):
+            first = max_ctx_len - m + 128 * qt
+            lo = max([0] + ([first - window + 1] if window else []) + ([first // chunk * chunk] if chunk else []))
+            pairs += min(max_ctx_len - 1, first + 127) // 128 - lo // 128 + 1
+    return min((1, 2, 4), key=lambda s: -(-max(1, pairs) * s // sm_count) * (TALK_START_BLOCKS + 8 / s))
+
+
 def talk_attention_prefill(q: torch.Tensor, q_col: int, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor, step,
                            n_heads: int, n_kv: int, head_dim: int, v_head_dim: int, window: Optional[int], chunk: Optional[int],
                            scale: float, cap: float, talk: Optional[torch.Tensor]) -> Optional[torch.Tensor]:
@@ -416,10 +431,7 @@ def talk_attention_prefill(q: torch.Tensor, q_col: int, k_cache: torch.Tensor, v
             [c_void_p, c_int64, c_int, c_void_p, c_void_p], defines)
     for qt0 in range(0, n_qt, at_once):
         n = min(at_once, n_qt - qt0)
-        # few (query tile, key tile) pairs: several CTAs share one (about half of the pairs of a causal prompt exist)
-        pairs, q_split = n_long * n * tiles, 1
-        while q_split < 4 and pairs * q_split < 2 * st.sm_count:
-            q_split *= 2
+        q_split = talk_q_split(st.sm_count, [m for m in step.seg_lens if m > 1], step.max_ctx_len, window, chunk, qt0, n)
         _call(f, q.data_ptr(), ld, int(q_col), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), block_table.data_ptr(),
               block_table.shape[1], step.seg_start.data_ptr(), step.seg_pos0.data_ptr(), step.seg_pos0.numel(), T, n_heads, n_kv, head_dim,
               v_head_dim, page_size, int(window or 0), int(chunk or 0), float(scale), float(cap or 0.0), _ptr(talk), n_pages, qt0, n, tiles,
