@@ -446,6 +446,7 @@ talk_split_kernel(const SplitArgs a) {
 
 // One CTA per (token, head), a thread per channel: the chunks' parts in ascending order, then the division.
 constexpr int MERGE_THREADS = 128;
+constexpr int MERGE_WEIGHTS = 1024;          // chunks whose weights are kept (65,536 keys; beyond that they are computed again)
 __global__ void __launch_bounds__(MERGE_THREADS)
 talk_merge_kernel(const float* __restrict__ parts, const int* __restrict__ token_seg, const int* __restrict__ positions,
                   const int* __restrict__ single_only, bf16* __restrict__ out, int H, int dv, int window, int chunk, int n_chunks) {
@@ -459,24 +460,27 @@ talk_merge_kernel(const float* __restrict__ parts, const int* __restrict__ token
     const int n = min(n_chunks, pos / KC - lo / KC + 1);
     const int64_t stride = dv + 2;
     const float* mine = parts + (t * H + h) * n_chunks * stride;
-    // every warp finds the maximum and the sum for itself
+    // every warp finds the maximum and the sum for itself; the chunks' weights go through shared memory
+    __shared__ float weight[MERGE_WEIGHTS];
     float m = -INFINITY;
     for (int i = lane; i < n; i += 32) m = fmaxf(m, mine[i * stride]);
     m = ib::warp_max(m);
     float l = 0.0f;
     for (int i = lane; i < n; i += 32) {
-        const float mi = mine[i * stride];
-        l += mi > -INFINITY ? mine[i * stride + 1] * expf(mi - m) : 0.0f;
+        const float mi = mine[i * stride], w = mi > -INFINITY ? expf(mi - m) : 0.0f;
+        l += mine[i * stride + 1] * w;
+        if (tid < 32 && i < MERGE_WEIGHTS) weight[i] = w;
     }
     l = ib::warp_sum(l);
     const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+    __syncthreads();
     for (int c = tid; c < dv; c += MERGE_THREADS) {
         float acc = 0.0f;
-#pragma unroll 4
-        for (int i = 0; i < n; i++) {
-            const float mi = mine[i * stride];
-            acc = fmaf(mine[i * stride + 2 + c], mi > -INFINITY ? expf(mi - m) : 0.0f, acc);
-        }
+        const float* col = mine + 2 + c;
+        const int n_s = min(n, MERGE_WEIGHTS);
+#pragma unroll 16
+        for (int i = 0; i < n_s; i++) acc = fmaf(col[i * stride], weight[i], acc);
+        for (int i = n_s; i < n; i++) acc = fmaf(col[i * stride], mine[i * stride] > -INFINITY ? expf(mine[i * stride] - m) : 0.0f, acc);
         out[(t * H + h) * dv + c] = __float2bfloat16_rn(acc * inv);
     }
 }

@@ -254,9 +254,14 @@ class HyperPreNormBlock(Block):
 
     def forward(self, h, step, cache, write_cache=True):
         dtype = self.mixer.rt.dtype
+        # In a decode step every kernel is a few microseconds of latency: a feed-forward with two independent chains of
+        # them (router beside the first product) may put one on a side stream.
+        side = _side_streams(h.device)[0] if (PARALLEL_BRANCHES and step.decode_only and dtype != torch.float32
+                                              and getattr(self.feed_forward, "takes_side_stream", False)) else None
         n = h.read(self.mixer_link, self.mixer_norm, dtype)
         h.write(self.mixer_link, self.mixer.forward(n, step, cache, None, write_cache))
         if self.feed_forward is not None:
             n = h.read(self.feed_forward_link, self.feed_forward_norm, dtype)
-            h.write(self.feed_forward_link, self.feed_forward.forward(n, None))
+            y = self.feed_forward.forward(n, None) if side is None else self.feed_forward.forward(n, None, side)
+            h.write(self.feed_forward_link, y)
         return h

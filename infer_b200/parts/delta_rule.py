@@ -191,8 +191,22 @@ class ChannelDeltaRule(GatedDeltaRule):
             self.filter_w = torch.cat([params[n["q_filter"]], params[n["k_filter"]], params[n["v_filter"]]], dim=0).to(**f32).t().contiguous()
 
     def forward(self, x, step, cache, residual, write_cache=True):
+        # In a decode step every kernel is a few microseconds of latency: the low-rank products run beside the others.
+        from .block import PARALLEL_BRANCHES, _side_streams
+        side = _side_streams(x.device)[1] if (PARALLEL_BRANCHES and step.decode_only and self.rt.dtype != torch.float32) else None
+        if side is not None:
+            main = torch.cuda.current_stream(x.device)
+            fork, done = torch.cuda.Event(), torch.cuda.Event()
+            fork.record(main)
+            side.wait_event(fork)
+            with torch.cuda.stream(side):
+                logits = self.up(self.low(x), out_dtype=torch.float32)
+                done.record(side)
         rows = self.proj(x, out_dtype=torch.float32)
-        logits = self.up(self.low(x), out_dtype=torch.float32)
+        if side is not None:
+            main.wait_event(done)
+        else:
+            logits = self.up(self.low(x), out_dtype=torch.float32)
         tails = cache.get("tails")
         inline_tail = tails is not None and write_cache and step.max_q_len == 1
         prep = ops.delta_prepare(rows, 0, 0, self.beta_col, self.filter_w, tails, self.a_log, self.dt_bias, self.unit_eps,

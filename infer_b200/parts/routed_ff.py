@@ -111,7 +111,24 @@ class RoutedExperts(FeedForward):
         self.down = Linear(self.rt, torch.cat([params[u + ".down"] for u in units], dim=1))
         self.width = E * self.ff + self.shared_ff
 
-    def forward(self, x, residual):
+    takes_side_stream = True
+
+    def forward(self, x, residual, side_stream=None):
+        """With ``side_stream`` the router runs there, beside the experts' first product (forked and joined here)."""
+        if side_stream is None:
+            return self._experts(self._weights(x), self.gate_up(x), residual)
+        main = torch.cuda.current_stream(x.device)
+        fork, done = torch.cuda.Event(), torch.cuda.Event()
+        fork.record(main)
+        side_stream.wait_event(fork)
+        with torch.cuda.stream(side_stream):
+            weights = self._weights(x)
+            done.record(side_stream)
+        rows = self.gate_up(x)
+        main.wait_event(done)
+        return self._experts(weights, rows, residual)
+
+    def _weights(self, x):
         logits = self.router(x, out_dtype=torch.float32)
         if self.router_kind == "sigmoid":
             weights, _ = ops.route_sigmoid(logits, self.correction, self.top, self.out_scale)
@@ -119,7 +136,9 @@ class RoutedExperts(FeedForward):
             weights, _ = ops.route(logits, self.top, self.groups, self.keep, sigmoid=True, group_best=2, renormalise=False, mult=self.out_scale)
         else:
             weights, _ = ops.route(logits, self.top, self.groups, self.keep, self.sum_eps)
-        rows = self.gate_up(x)
+        return weights
+
+    def _experts(self, weights, rows, residual):
         if self.expert_kind == "relu_squared":
             if self.shared_ff:
                 raise NotImplementedError("a shared expert of the relu_squared form")
