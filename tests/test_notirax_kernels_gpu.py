@@ -318,7 +318,7 @@ def test_delta_rule_with_decays_per_channel_over_steps(sizes, taps):
 
 # ----------------------------------------------------------------------------------------------- the router
 
-@pytest.mark.parametrize("E,top,count,keep", [(16, 2, 2, 1), (8, 8, 1, 1), (12, 3, 4, 2), (6, 2, 6, 3), (40, 6, 5, 5), (64, 4, 8, 3), (1, 1, 1, 1)])
+@pytest.mark.parametrize("E,top,count,keep", [(20, 3, 2, 1), (8, 8, 1, 1), (12, 3, 4, 2), (6, 2, 6, 3), (40, 6, 5, 5), (64, 4, 8, 3), (1, 1, 1, 1)])
 def test_router_with_sigmoid_scores_and_groups_of_two_best(E, top, count, keep):
     g = torch.Generator().manual_seed(E + top)
     logits = 2.0 * torch.randn(65, E, generator=g)
