@@ -34,6 +34,7 @@ MODULES: Dict[str, str] = {
     "latent": "latent_ops.cu",   # attention through low-rank latents, layer norm, sigmoid router, capped logits
     "post": "post_ops.cu",       # norms after the residual sum, per-head query/key norms, mixtures with the token before
     "stream": "stream_ops.cu",   # several residual streams, norms over groups of channels, sinusoidal positions
+    "memory": "memory_ops.cu",   # scaled sums with the next norm, state space layers' filters and steps, matrix memories' gates
     "talk": "talk_ops.cu",       # attention whose heads exchange their scores before the softmax
     "talk_pf": "talk_prefill.cu",       # the same attention for prompt portions on the tensor cores
     "latent_pf": "latent_prefill.cu",   # the same attention for prompt portions: per-head keys and values, tensor cores

@@ -1,0 +1,308 @@
+// Kernels for layers whose sublayers' results enter the residual stream through a factor per channel, for state space
+// layers (a filter over time in front of a matrix state that fades by one number per head and token) and for matrix
+// memories with exponential gates. The recurrences themselves are state_scan mode 5 (mix_ops.cu).
+//
+// Rows of recurrences, the residual stream and all arithmetic are float; the normalised rows that a layer's first matrix
+// products read leave in float or bfloat16. With float storage these kernels are the 32-bit path.
+//
+// A step's rows are the tokens of several requests ("segments") one after the other: seg_start[s] is the first row
+// of segment s, seg_slot[s] the request's state slot. A token's result depends on its own request's earlier tokens
+// and state only, and every sum runs in an order fixed by the layer's sizes.
+#include "common.cuh"
+
+IB_DEFINE_LAST_ERROR()
+
+#define IB_LAUNCH(kernel, grid, block, smem, ...)                                                              \
+    do {                                                                                                       \
+        const int rc_ = ib::launch(#kernel, kernel, dim3(grid), dim3(block), size_t(smem), stream, 1u, __VA_ARGS__); \
+        if (rc_) return rc_;                                                                                   \
+    } while (0)
+
+namespace {
+
+using bf16 = __nv_bfloat16;
+
+inline unsigned blocks_for(int64_t n, int threads) { return unsigned((n + threads - 1) / threads); }
+
+__device__ __forceinline__ float silu_(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float softplus_(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
+__device__ __forceinline__ float log_sigmoid_(float x) { return fminf(x, 0.0f) - log1pf(expf(-fabsf(x))); }
+
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(bf16* p, float4 v) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    uint2 u;
+    u.x = *reinterpret_cast<unsigned*>(&lo);
+    u.y = *reinterpret_cast<unsigned*>(&hi);
+    *reinterpret_cast<uint2*>(p) = u;
+}
+
+// ------------------------------------------------------------------------------------------------
+// y = x + wa * a + wb * b per row (a, b may be absent; wa, wb: a factor per channel), kept in x with `store`; then
+// out = y / sqrt(mean(y^2) + eps) * w, the rows the next sublayers read. `rows` picks and orders input rows (nothing is
+// stored then). One CTA per row. VEC: four channels a thread and access.
+template <typename TOut, int VEC>
+__global__ void __launch_bounds__(256)
+scaled_sum_norm_kernel(float* __restrict__ x, const float* __restrict__ a, const float* __restrict__ wa, const float* __restrict__ b,
+                       const float* __restrict__ wb, const float* __restrict__ w, float eps, const int* __restrict__ rows, int store,
+                       TOut* __restrict__ out, int64_t width) {
+    __shared__ float red[32];
+    ib::pdl_launch_dependents();
+    ib::pdl_wait();
+    const int64_t t = rows ? rows[blockIdx.x] : blockIdx.x;
+    float* xr = x + t * width;
+    const float* ar = a ? a + t * width : nullptr;
+    const float* br = b ? b + t * width : nullptr;
+    TOut* o = out + int64_t(blockIdx.x) * width;
+    auto sum1 = [&](int64_t i) {
+        float y = xr[i];
+        if (ar) y = fmaf(wa[i], ar[i], y);
+        if (br) y = fmaf(wb[i], br[i], y);
+        return y;
+    };
+    float ss = 0.0f;
+    if (VEC == 4) {
+        // a thread keeps its first row pieces in registers (rows of up to KEEP * 1024 channels whole)
+        constexpr int KEEP = 4;
+        float4 kept[KEEP];
+        int n = 0;
+        auto sum4 = [&](int64_t i) {
+            float4 y = load4(xr + i);
+            if (ar) {
+                const float4 f = load4(wa + i), v = load4(ar + i);
+                y.x = fmaf(f.x, v.x, y.x); y.y = fmaf(f.y, v.y, y.y); y.z = fmaf(f.z, v.z, y.z); y.w = fmaf(f.w, v.w, y.w);
+            }
+            if (br) {
+                const float4 f = load4(wb + i), v = load4(br + i);
+                y.x = fmaf(f.x, v.x, y.x); y.y = fmaf(f.y, v.y, y.y); y.z = fmaf(f.z, v.z, y.z); y.w = fmaf(f.w, v.w, y.w);
+            }
+            return y;
+        };
+#pragma unroll
+        for (int k = 0; k < KEEP; k++) {
+            const int64_t i = (int64_t(k) * blockDim.x + threadIdx.x) * 4;
+            if (i < width) {
+                kept[k] = sum4(i);
+                n = k + 1;
+                ss = fmaf(kept[k].x, kept[k].x, ss); ss = fmaf(kept[k].y, kept[k].y, ss);
+                ss = fmaf(kept[k].z, kept[k].z, ss); ss = fmaf(kept[k].w, kept[k].w, ss);
+            }
+        }
+        for (int64_t i = (int64_t(KEEP) * blockDim.x + threadIdx.x) * 4; i < width; i += int64_t(blockDim.x) * 4) {
+            const float4 y = sum4(i);
+            ss = fmaf(y.x, y.x, ss); ss = fmaf(y.y, y.y, ss); ss = fmaf(y.z, y.z, ss); ss = fmaf(y.w, y.w, ss);
+        }
+        ss = ib::block_sum(ss, red);
+        const float f = 1.0f / sqrtf(ss / float(width) + eps);
+        auto finish = [&](int64_t i, float4 y) {
+            if (store && ar) store4(xr + i, y);
+            const float4 wv = load4(w + i);
+            store4(o + i, make_float4(y.x * f * wv.x, y.y * f * wv.y, y.z * f * wv.z, y.w * f * wv.w));
+        };
+#pragma unroll
+        for (int k = 0; k < KEEP; k++)
+            if (k < n) finish((int64_t(k) * blockDim.x + threadIdx.x) * 4, kept[k]);
+        for (int64_t i = (int64_t(KEEP) * blockDim.x + threadIdx.x) * 4; i < width; i += int64_t(blockDim.x) * 4) finish(i, sum4(i));
+        return;
+    }
+    for (int64_t i = threadIdx.x; i < width; i += blockDim.x) {
+        const float y = sum1(i);
+        ss = fmaf(y, y, ss);
+    }
+    ss = ib::block_sum(ss, red);
+    const float f = 1.0f / sqrtf(ss / float(width) + eps);
+    for (int64_t i = threadIdx.x; i < width; i += blockDim.x) {
+        const float y = sum1(i);
+        if (store && ar) xr[i] = y;
+        o[i] = ib::from_f32<TOut>(y * f * w[i]);
+    }
+}
+
+// ------------------------------------------------------------------------------------------------
+// What a state space layer's recurrence reads, from the projected rows: columns [col0, col0 + channels) each through a
+// causal filter over time, y_t = bias + sum_j w[j][c] u_(t - taps + 1 + j) (u before the segment's first row comes from
+// the request's tail, its last taps - 1 inputs, oldest first; zeros for a new request), then silu; and per head, from
+// column dt_col, dt = softplus(raw + dt_bias[h]) and g = exp(-exp(a_log[h]) dt).
+// out rows (ldo): [channels | up to a multiple of 4 | g (H) | dt (H)]. Filter weights tap-major [taps, channels].
+// inline_tail (steps of one token per request only): the thread that filters a channel, the only reader of its tail, moves it.
+// A CTA of 128 threads: VEC channels a thread, grid (tokens, blocks of channels and heads).
+template <int VEC>
+__global__ void __launch_bounds__(128)
+filter_prepare_kernel(const float* __restrict__ rows, int64_t ld, int col0, int channels, const float* __restrict__ filt_w,
+                      const float* __restrict__ filt_b, int taps, float* tails, int inline_tail, int dt_col,
+                      const float* __restrict__ dt_bias, const float* __restrict__ a_log, int n_heads, const int* __restrict__ token_seg,
+                      const int* __restrict__ seg_start, const int* __restrict__ seg_slot, float* __restrict__ out, int64_t ldo) {
+    ib::pdl_launch_dependents();
+    ib::pdl_wait();
+    const int64_t t = blockIdx.x;
+    const int u = blockIdx.y * blockDim.x + threadIdx.x;
+    const int n_units = (channels + VEC - 1) / VEC;
+    if (u >= n_units) {
+        const int h = u - n_units;
+        if (h >= n_heads) return;
+        const float dt = softplus_(rows[t * ld + dt_col + h] + dt_bias[h]);
+        float* o = out + t * ldo + (channels + 3) / 4 * 4;
+        o[h] = expf(-expf(a_log[h]) * dt);
+        o[n_heads + h] = dt;
+        return;
+    }
+    const int c = u * VEC;
+    const int s = token_seg[t];
+    const int i_local = int(t - seg_start[s]);
+    float* tail = taps > 1 ? tails + int64_t(seg_slot[s]) * (taps - 1) * channels + c : nullptr;
+    float y[VEC], newest[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; e++) { y[e] = filt_b[c + e]; newest[e] = 0.0f; }
+    for (int j = 0; j < taps; j++) {
+        const int back = taps - 1 - j;
+        const float* in = i_local >= back ? rows + (t - back) * ld + col0 + c : tail + int64_t(taps - 1 + i_local - back) * channels;
+        const float* w = filt_w + int64_t(j) * channels + c;
+        if (VEC == 4) {
+            const float4 v = load4(in), f = load4(w);
+            y[0] = fmaf(f.x, v.x, y[0]); y[1 % VEC] = fmaf(f.y, v.y, y[1 % VEC]);
+            y[2 % VEC] = fmaf(f.z, v.z, y[2 % VEC]); y[3 % VEC] = fmaf(f.w, v.w, y[3 % VEC]);
+            newest[0] = v.x; newest[1 % VEC] = v.y; newest[2 % VEC] = v.z; newest[3 % VEC] = v.w;
+        } else {
+            newest[0] = in[0];
+            y[0] = fmaf(w[0], newest[0], y[0]);
+        }
+    }
+    if (inline_tail && taps > 1) {
+        for (int idx = 0; idx + 1 < taps - 1; idx++)
+#pragma unroll
+            for (int e = 0; e < VEC; e++) tail[int64_t(idx) * channels + e] = tail[int64_t(idx + 1) * channels + e];
+#pragma unroll
+        for (int e = 0; e < VEC; e++) tail[int64_t(taps - 2) * channels + e] = newest[e];
+    }
+    float* o = out + t * ldo + c;
+    if (VEC == 4) {
+        store4(o, make_float4(silu_(y[0]), silu_(y[1 % VEC]), silu_(y[2 % VEC]), silu_(y[3 % VEC])));
+    } else {
+        o[0] = silu_(y[0]);
+    }
+}
+
+// ------------------------------------------------------------------------------------------------
+// Gates of a matrix memory over the tokens of every segment in order, one CTA per (segment, head):
+//   i = cap tanh((raw[i_col + h] + i_bias[h]) / cap),   f = log sigmoid(cap tanh((raw[f_col + h] + f_bias[h]) / cap))
+//   m <- max(f + m, i)   (m kept per request and head in `state` [slots, H], zero for a new request)
+//   out rows (ldo): [keep = exp(f + m_before - m) (H) | write = exp(i - m) (H) | floor = exp(-m) (H)]
+// The gates and the exponentials are computed in parallel over a tile of tokens; the running maximum walks the tile in
+// one thread, an addition and a maximum a token, so that it does not depend on where a prompt was cut.
+constexpr int GATE_TILE = 512;
+
+__global__ void __launch_bounds__(128)
+memory_gates_kernel(const float* __restrict__ rows, int64_t ld, int i_col, int f_col, const float* __restrict__ i_bias,
+                    const float* __restrict__ f_bias, float cap, float* __restrict__ state, const int* __restrict__ seg_start,
+                    const int* __restrict__ seg_slot, float* __restrict__ out, int64_t ldo, int n_heads, int write_state) {
+    __shared__ __align__(16) float gi[GATE_TILE], gf[GATE_TILE], gm[GATE_TILE + 4];
+    ib::pdl_launch_dependents();
+    ib::pdl_wait();
+    const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+    const int64_t t0 = seg_start[s];
+    const int len = int(seg_start[s + 1] - t0);
+    float* kept = state + int64_t(seg_slot[s]) * n_heads + h;
+    const float bi = i_bias[h], bf = f_bias[h];
+    float m = *kept;
+    for (int c0 = 0; c0 < len; c0 += GATE_TILE) {
+        const int n = min(GATE_TILE, len - c0);
+        for (int c = tid; c < n; c += blockDim.x) {
+            const float* r = rows + (t0 + c0 + c) * ld;
+            gi[c] = cap * tanhf((r[i_col + h] + bi) / cap);
+            gf[c] = log_sigmoid_(cap * tanhf((r[f_col + h] + bf) / cap));
+        }
+        __syncthreads();
+        if (tid == 0) {
+            // gm[c] is the maximum before token c, gm[n] the one after the tile
+            int c = 0;
+            for (; c + 4 <= n; c += 4) {
+                const float4 i4 = load4(gi + c), f4 = load4(gf + c);
+                float4 b4;
+                b4.x = m;
+                m = fmaxf(f4.x + m, i4.x);
+                b4.y = m;
+                m = fmaxf(f4.y + m, i4.y);
+                b4.z = m;
+                m = fmaxf(f4.z + m, i4.z);
+                b4.w = m;
+                m = fmaxf(f4.w + m, i4.w);
+                store4(gm + c, b4);
+            }
+            for (; c < n; c++) {
+                gm[c] = m;
+                m = fmaxf(gf[c] + m, gi[c]);
+            }
+            gm[n] = m;
+        }
+        __syncthreads();
+        for (int c = tid; c < n; c += blockDim.x) {
+            float* o = out + (t0 + c0 + c) * ldo;
+            const float now = gm[c + 1];
+            o[h] = expf(gf[c] + gm[c] - now);
+            o[n_heads + h] = expf(gi[c] - now);
+            o[2 * n_heads + h] = expf(-now);
+        }
+        m = gm[n];
+        __syncthreads();
+    }
+    if (write_state && tid == 0) *kept = m;
+}
+
+}  // namespace
+
+// ================================================================================================
+// C entry points. dtype arguments: 0 = float, 1 = bfloat16.
+
+IB_EXPORT int ib_scaled_sum_norm(float* x, const float* a, const float* wa, const float* b, const float* wb, const float* w, float eps,
+                                 const int* rows, int store, void* out, int out_dtype, int64_t n_rows, int64_t width,
+                                 cudaStream_t stream) {
+    if (n_rows <= 0 || width <= 0) return IB_OK;
+    if (!x || !w || !out || (a && !wa) || (b && (!wb || !a))) return ib::fail(IB_ERR_ARG, "ib_scaled_sum_norm: rows, their factors and a weight are needed");
+    if (rows) store = 0;
+    const uintptr_t all = uintptr_t(x) | uintptr_t(a) | uintptr_t(wa) | uintptr_t(b) | uintptr_t(wb) | uintptr_t(w) | uintptr_t(out);
+    const bool vec = width % 4 == 0 && !(all & 15);           // (by sizes and addresses, never by the number of rows)
+#define IB_SSN(TO, VV) IB_LAUNCH((scaled_sum_norm_kernel<TO, VV>), unsigned(n_rows), 256, 0, x, a, wa, b, wb, w, eps, rows, store, (TO*)out, width)
+    if (out_dtype == IB_F32) {
+        if (vec) IB_SSN(float, 4); else IB_SSN(float, 1);
+    } else if (out_dtype == IB_BF16) {
+        if (vec) IB_SSN(bf16, 4); else IB_SSN(bf16, 1);
+    } else {
+        return ib::fail(IB_ERR_ARG, "ib_scaled_sum_norm: unknown dtype %d", out_dtype);
+    }
+#undef IB_SSN
+    return ib::check_launch("ib_scaled_sum_norm");
+}
+
+IB_EXPORT int ib_filter_prepare(const float* rows, int64_t ld, int col0, int channels, const float* filt_w, const float* filt_b, int taps,
+                                float* tails, int inline_tail, int dt_col, const float* dt_bias, const float* a_log, int n_heads,
+                                const int* token_seg, const int* seg_start, const int* seg_slot, float* out, int64_t ldo,
+                                int64_t n_tokens, cudaStream_t stream) {
+    if (n_tokens <= 0) return IB_OK;
+    if (channels <= 0 || taps <= 0 || n_heads <= 0 || !filt_w || !filt_b) return ib::fail(IB_ERR_ARG, "ib_filter_prepare: bad sizes");
+    if (taps > 1 && !tails) return ib::fail(IB_ERR_ARG, "ib_filter_prepare: a filter of %d taps needs tails", taps);
+    if (ldo < (channels + 3) / 4 * 4 + 2 * int64_t(n_heads)) return ib::fail(IB_ERR_ARG, "ib_filter_prepare: result rows too short");
+    const uintptr_t all = uintptr_t(rows) | uintptr_t(filt_w) | uintptr_t(taps > 1 ? tails : nullptr) | uintptr_t(out);
+    const bool vec = channels % 4 == 0 && col0 % 4 == 0 && ld % 4 == 0 && ldo % 4 == 0 && !(all & 15);
+    const int units = (vec ? channels / 4 : channels) + n_heads;
+    const dim3 grid{unsigned(n_tokens), blocks_for(units, 128), 1u};
+    if (grid.y > 65535) return ib::fail(IB_ERR_ARG, "ib_filter_prepare: too many channels");
+    if (vec)
+        IB_LAUNCH(filter_prepare_kernel<4>, grid, 128, 0, rows, ld, col0, channels, filt_w, filt_b, taps, tails, inline_tail, dt_col, dt_bias,
+                  a_log, n_heads, token_seg, seg_start, seg_slot, out, ldo);
+    else
+        IB_LAUNCH(filter_prepare_kernel<1>, grid, 128, 0, rows, ld, col0, channels, filt_w, filt_b, taps, tails, inline_tail, dt_col, dt_bias,
+                  a_log, n_heads, token_seg, seg_start, seg_slot, out, ldo);
+    return ib::check_launch("ib_filter_prepare");
+}
+
+IB_EXPORT int ib_memory_gates(const float* rows, int64_t ld, int i_col, int f_col, const float* i_bias, const float* f_bias, float cap,
+                              float* state, const int* seg_start, const int* seg_slot, float* out, int64_t ldo, int n_segments,
+                              int n_heads, int write_state, cudaStream_t stream) {
+    if (n_segments <= 0) return IB_OK;
+    if (n_heads <= 0 || n_heads > 65535 || !(cap > 0.0f) || ldo < 3 * int64_t(n_heads))
+        return ib::fail(IB_ERR_ARG, "ib_memory_gates: %d heads, a cap of %f", n_heads, double(cap));
+    IB_LAUNCH(memory_gates_kernel, (dim3{unsigned(n_segments), unsigned(n_heads), 1u}), 128, 0, rows, ld, i_col, f_col, i_bias, f_bias, cap,
+              state, seg_start, seg_slot, out, ldo, n_heads, write_state);
+    return ib::check_launch("ib_memory_gates");
+}

@@ -543,13 +543,14 @@ split_attention_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
 }
 
 // One warp per (token, head): the chunks' parts in ascending order, the sink, the division; optionally times
-// sigmoid(gate[t, gate_col + h dv + c]) (the logits of a gate per output channel, rows of leading dimension ldg).
+// sigmoid(gate[t, gate_col + h dv + c]) (the logits of a gate per output channel, rows of leading dimension ldg), or with
+// `gate_per_head` sigmoid(gate[t, gate_col + h]).
 template <typename T>
 __global__ void split_attention_merge_kernel(const float* __restrict__ parts, const int* __restrict__ token_seg,
                                              const int* __restrict__ positions, const int* __restrict__ single_only,
                                              const float* __restrict__ sink, T* __restrict__ out, int64_t n_rows, int n_heads,
                                              int dv, int window, int n_chunks, int keep_first, const T* __restrict__ gate,
-                                             int64_t ldg, int64_t gate_col) {
+                                             int64_t ldg, int64_t gate_col, int gate_per_head) {
     ib::pdl_wait();
     const int lane = threadIdx.x & 31;
     const int64_t r = int64_t(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -595,8 +596,8 @@ __global__ void split_attention_merge_kernel(const float* __restrict__ parts, co
             if (c >= dv) continue;
             const float o = acc[e];
         float y = o * inv;
-        // (a gate per output channel: the result is rounded as the ungated kernel leaves it, then multiplied)
-        if (gate) y = ib::to_f32(ib::from_f32<T>(y)) * sigmoid_(ib::to_f32(gate[t * ldg + gate_col + int64_t(h) * dv + c]));
+        // (a gate: the result is rounded as the ungated kernel leaves it, then multiplied)
+        if (gate) y = ib::to_f32(ib::from_f32<T>(y)) * sigmoid_(ib::to_f32(gate[t * ldg + gate_col + (gate_per_head ? int64_t(h) : int64_t(h) * dv + c)]));
         out[r * dv + c] = ib::from_f32<T>(y);
         }
     }
@@ -766,11 +767,16 @@ __global__ void tail_update_kernel(const float* __restrict__ rows, int64_t ld, i
 //                                       o_t = (S + diag(u) k_t v_t^T)^T q_t;  then  S <- diag(a_t) S + k_t v_t^T
 //   MODE 4 (delta rule, a decay per key channel):
 //                                       S <- diag(a_t) S;  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t
+//   MODE 5 (a decay and a write strength per head and token):
+//                                       S <- g_t S + beta_t k_t v_t^T;               o_t = S^T q_t + skip_h v_t
 // MODE 1 is computed from the old state in one sweep: r = S^T k, p = S^T q, u = beta (v - g r), o = g p + u (k.q),
 // S <- g S + k u^T, with k.q given per token (aux rows). MODE 2 reads g at aux_col + h of the token's aux row (a
 // leading dimension of 0: one row for every token). MODE 3 reads its decays as MODE 0 and u [heads, d] from `bonus`.
 // MODE 4 reads its decays as MODE 0, beta at scal_col + h and k.q at scal_col + H + h / heads_per_qk of the same aux
 // rows, and works in one sweep as MODE 1: S <- diag(a) S with r = S^T k and p = S^T q, then S <- S + k u^T, o = p + u (k.q).
+// MODE 5 reads g at aux_col + h and beta at aux_col + H + h, and skip [heads] from `bonus` (null: none). With `ones_state`
+// [slots, heads, d] it runs one more column whose values are all 1, n <- g n + beta k, kept there, and its read-out n.q goes
+// to ones_out [tokens, heads] (what a read-out is normalised by).
 // A column of S belongs to LK = 8 neighbouring lanes, lane j of them keeping rows j R .. j R + R - 1 in registers
 // (R >= d / 8, rows beyond d are zero and stay zero); a warp has 4 columns, a CTA `cb` columns of one (segment, head).
 // Column sums are added within a lane in four chains and across the 8 lanes by shuffles, in an order that depends on
@@ -803,7 +809,7 @@ struct ScanOperands {
 #pragma unroll
             for (int i = 0; i < R / 4; i++) a[i] = a4[i];
         }
-        if (MODE == 1 || MODE == 2 || MODE == 4) { g = ss[c * 4 + 0]; beta = ss[c * 4 + 1]; kq = ss[c * 4 + 2]; }
+        if (MODE == 1 || MODE == 2 || MODE == 4 || MODE == 5) { g = ss[c * 4 + 0]; beta = ss[c * 4 + 1]; kq = ss[c * 4 + 2]; }
         v = vs[c * cb + col_l];
     }
 };
@@ -811,8 +817,8 @@ struct ScanOperands {
 // One token through a thread's share of the state; returns the column's read-out (valid in every lane of its group).
 template <int R, int MODE>
 __device__ __forceinline__ float scan_token(float (&S)[R], const ScanOperands<R, MODE>& x, const float* U) {
-    const float v = x.v;
-    if (MODE == 2) {
+    const float v = MODE == 5 ? x.beta * x.v : x.v;
+    if (MODE == 2 || MODE == 5) {
         const float g = x.g;
         float p0 = 0.0f, p1 = 0.0f, p2 = 0.0f, p3 = 0.0f;
 #pragma unroll
@@ -954,12 +960,12 @@ state_scan_kernel(const float* __restrict__ rows, int64_t ld, int q_col, int k_c
                   const float* __restrict__ aux, int64_t lda, int aux_col, float* __restrict__ state,
                   const int* __restrict__ seg_start, const int* __restrict__ seg_slot, float* __restrict__ raw_out,
                   int n_heads, int heads_per_qk, int d, int dv, int cb, int chunk, int write_state, int pipelined,
-                  const float* __restrict__ bonus, int act, int scal_col) {
+                  const float* __restrict__ bonus, int act, int scal_col, float* __restrict__ ones_state, float* __restrict__ ones_out) {
     extern __shared__ __align__(16) float sm[];
     constexpr int RP = R + 4, DPP = LK * RP;
     constexpr bool ROWS = MODE == 0 || MODE == 3 || MODE == 4;      // the decays are rows like q and k
-    constexpr bool SCAL = MODE == 1 || MODE == 2 || MODE == 4;      // scalars per token: [g, beta, k.q] in places 0..2
-    constexpr int SCAL0 = MODE == 4 ? 1 : 0, SCAL1 = MODE == 2 ? 1 : 3;     // the places that this mode has
+    constexpr bool SCAL = MODE == 1 || MODE == 2 || MODE == 4 || MODE == 5;      // scalars per token: [g, beta, k.q] in places 0..2
+    constexpr int SCAL0 = MODE == 4 ? 1 : 0, SCAL1 = MODE == 2 ? 1 : (MODE == 5 ? 2 : 3);     // the places that this mode has
     const int n_buf = pipelined ? 2 : 1;
     const int a_tok = ROWS ? DPP : 0, s_tok = SCAL ? 4 : 0;
     float* qs = sm;                          // [n_buf][chunk][DPP]
@@ -972,16 +978,24 @@ state_scan_kernel(const float* __restrict__ rows, int64_t ld, int q_col, int k_c
     const int hq = h / heads_per_qk;
     const int lk = tid & (LK - 1), col_l = tid >> 3;
     const int col0 = blockIdx.z * cb, col = col0 + col_l;
-    const bool live = col < dv;
+    const bool ones = MODE == 5 && ones_state && col == dv;      // the column of ones behind the values
+    const bool live = col < dv || ones;
     const int k0 = lk * R, off = lk * RP;
     for (int i = tid; i < total; i += blockDim.x) sm[i] = 0.0f;       // padding and rows beyond d stay zero
+    if (MODE == 5 && ones_state && dv >= col0 && dv < col0 + cb) {
+        __syncthreads();
+        for (int i = tid; i < n_buf * chunk; i += blockDim.x) vs[i * cb + dv - col0] = 1.0f;
+    }
     ib::pdl_wait();
     const int64_t t0 = seg_start[s];
     const int len = int(seg_start[s + 1] - t0);
-    float* S_g = state + (int64_t(seg_slot[s]) * n_heads + h) * int64_t(d) * dv;
+    const int64_t s_row = ones ? 1 : dv;     // from one row of the thread's column to the next
+    float* S_g = ones ? ones_state + (int64_t(seg_slot[s]) * n_heads + h) * int64_t(d)
+                      : state + (int64_t(seg_slot[s]) * n_heads + h) * int64_t(d) * dv + col;
     float S[R];
 #pragma unroll
-    for (int i = 0; i < R; i++) S[i] = (live && k0 + i < d) ? S_g[int64_t(k0 + i) * dv + col] : 0.0f;
+    for (int i = 0; i < R; i++) S[i] = (live && k0 + i < d) ? S_g[int64_t(k0 + i) * s_row] : 0.0f;
+    const float skip = (MODE == 5 && bonus && !ones) ? bonus[h] : 0.0f;
     float U[MODE == 3 ? R : 1];
     if (MODE == 3) {
 #pragma unroll
@@ -1036,8 +1050,8 @@ state_scan_kernel(const float* __restrict__ rows, int64_t ld, int q_col, int k_c
         }
         for (int idx = tid; idx < n * cb; idx += blockDim.x) {
             const int c = idx / cb, j = col0 + (idx - c * cb);
-            const float vv = j < dv ? rows[(t0 + c0 + c) * ld + v_col + h * dv + j] : 0.0f;
-            vs[idx] = act ? silu_(vv) : vv;
+            const float vv = j < dv ? rows[(t0 + c0 + c) * ld + v_col + h * dv + j] : (MODE == 5 && ones_state && j == dv ? 1.0f : 0.0f);
+            vs[idx] = act && j < dv ? silu_(vv) : vv;
         }
     };
 
@@ -1065,8 +1079,13 @@ state_scan_kernel(const float* __restrict__ rows, int64_t ld, int q_col, int k_c
         cur.load(qb, kb, ab, sb, vb, 0, DPP, off, cb, col_l);
         for (int c = 0; c < n; c++) {
             if (c + 1 < n) nxt.load(qb, kb, ab, sb, vb, c + 1, DPP, off, cb, col_l);
-            const float o = scan_token<R, MODE>(S, cur, U);
-            if (lk == 0 && live) raw_out[((t0 + c0 + c) * n_heads + h) * int64_t(dv) + col] = o;
+            float o = scan_token<R, MODE>(S, cur, U);
+            if (MODE == 5) o = fmaf(skip, cur.v, o);
+            if (lk == 0 && live) {
+                const int64_t row = (t0 + c0 + c) * n_heads + h;
+                if (MODE == 5 && ones) ones_out[row] = o;
+                else raw_out[row * int64_t(dv) + col] = o;
+            }
             cur = nxt;
         }
         __syncthreads();                     // every thread has read this buffer: the copies after next may fill it
@@ -1075,7 +1094,7 @@ state_scan_kernel(const float* __restrict__ rows, int64_t ld, int q_col, int k_c
     if (write_state && live) {
 #pragma unroll
         for (int i = 0; i < R; i++)
-            if (k0 + i < d) S_g[int64_t(k0 + i) * dv + col] = S[i];
+            if (k0 + i < d) S_g[int64_t(k0 + i) * s_row] = S[i];
     }
 }
 
@@ -1212,7 +1231,7 @@ IB_EXPORT int ib_attention_split(const void* q, const void* k_cache, const void*
                                  int64_t n_tokens, int n_heads, int n_kv, int d, int dv, int page_size, int window, float scale,
                                  int64_t n_pages, const float* dist_bias, int bias_len, const float* sink, int visible, int dtype,
                                  int* status, cudaStream_t stream, int keep_first, const float* slopes, const void* gate, int64_t ldg,
-                                 int64_t gate_col) {
+                                 int64_t gate_col, int gate_per_head) {
     if (n_tokens <= 0) return IB_OK;
     if (n_kv <= 0 || n_heads % n_kv || n_heads / n_kv > GMAX)
         return ib::fail(IB_ERR_ARG, "ib_attention_split: %d heads on %d kv heads (groups of up to %d)", n_heads, n_kv, GMAX);
@@ -1245,11 +1264,11 @@ IB_EXPORT int ib_attention_split(const void* q, const void* k_cache, const void*
     if (dtype == IB_F32) {
         IB_SPLIT_BY_GROUP(float);
         IB_LAUNCH(split_attention_merge_kernel<float>, blocks_for(rows, 4), 128, 0, workspace, token_seg, positions, single_only, sink,
-                  (float*)out, rows, n_heads, dv, window, n_chunks, keep_first, (const float*)gate, ldg, gate_col);
+                  (float*)out, rows, n_heads, dv, window, n_chunks, keep_first, (const float*)gate, ldg, gate_col, gate_per_head);
     } else if (dtype == IB_BF16) {
         IB_SPLIT_BY_GROUP(bf16);
         IB_LAUNCH(split_attention_merge_kernel<bf16>, blocks_for(rows, 4), 128, 0, workspace, token_seg, positions, single_only, sink,
-                  (bf16*)out, rows, n_heads, dv, window, n_chunks, keep_first, (const bf16*)gate, ldg, gate_col);
+                  (bf16*)out, rows, n_heads, dv, window, n_chunks, keep_first, (const bf16*)gate, ldg, gate_col, gate_per_head);
     } else {
         return ib::fail(IB_ERR_ARG, "ib_attention_split: unknown dtype %d", dtype);
     }
@@ -1306,33 +1325,37 @@ template <int R, int MODE>
 static int launch_scan(dim3 grid, int threads, size_t smem, cudaStream_t stream, const float* rows, int64_t ld, int q_col,
                        int k_col, int v_col, const float* aux, int64_t lda, int aux_col, float* state, const int* seg_start,
                        const int* seg_slot, float* raw_out, int n_heads, int hpq, int d, int dv, int cb, int chunk, int write_state,
-                       int pipelined, const float* bonus, int act, int scal_col) {
+                       int pipelined, const float* bonus, int act, int scal_col, float* ones_state, float* ones_out) {
     IB_LAUNCH((state_scan_kernel<R, MODE>), grid, threads, smem, rows, ld, q_col, k_col, v_col, aux, lda, aux_col, state, seg_start,
-              seg_slot, raw_out, n_heads, hpq, d, dv, cb, chunk, write_state, pipelined, bonus, act, scal_col);
+              seg_slot, raw_out, n_heads, hpq, d, dv, cb, chunk, write_state, pipelined, bonus, act, scal_col, ones_state, ones_out);
     return ib::check_launch("ib_state_scan");
 }
 
 // mode 0: a decay per key channel (aux: decays at aux_col + h d); mode 1: gated delta rule (aux: g, beta, k.q);
 // mode 2: a decay per head (aux: at aux_col + h; lda 0: the same for every token); mode 3: as mode 0 with the read-out
 // before the write and `bonus` [heads, d] on the current token; mode 4: delta rule with decays as mode 0 and beta, k.q at
-// scal_col of the aux rows.
+// scal_col of the aux rows; mode 5: a decay and a write strength per head and token (aux: at aux_col + h and aux_col + H + h),
+// skip [heads] in `bonus` (null: none), with ones_state and ones_out a column of ones beside the values.
 // `spread` (prompt portions): a head's columns go to more, smaller CTAs until there is about one per SM (sm_count).
 IB_EXPORT int ib_state_scan(int mode, const float* rows, int64_t ld, int q_col, int k_col, int v_col, const float* aux,
                             int64_t lda, int aux_col, float* state, const int* seg_start, const int* seg_slot,
                             float* raw_out, int n_segments, int n_heads, int heads_per_qk, int d, int dv, int write_state,
-                            int spread, int sm_count, cudaStream_t stream, const float* bonus, int act, int scal_col) {
+                            int spread, int sm_count, cudaStream_t stream, const float* bonus, int act, int scal_col,
+                            float* ones_state, float* ones_out) {
     if (n_segments <= 0) return IB_OK;
     if (n_heads <= 0 || n_heads > 65535 || heads_per_qk <= 0 || n_heads % heads_per_qk || d <= 0 || dv <= 0 || d > LK * 32)
         return ib::fail(IB_ERR_ARG, "ib_state_scan: %d heads with a state of %d x %d do not fit", n_heads, d, dv);
-    if (mode < 0 || mode > 4) return ib::fail(IB_ERR_ARG, "ib_state_scan: unknown mode %d", mode);
+    if (mode < 0 || mode > 5) return ib::fail(IB_ERR_ARG, "ib_state_scan: unknown mode %d", mode);
     if (mode == 3 && !bonus) return ib::fail(IB_ERR_ARG, "ib_state_scan: mode 3 needs the bonus");
+    if (ones_state && (mode != 5 || !ones_out)) return ib::fail(IB_ERR_ARG, "ib_state_scan: a column of ones goes with mode 5 and a result of its own");
     const bool decay_rows = mode == 0 || mode == 3 || mode == 4;
+    const int columns = dv + (ones_state ? 1 : 0);
     const int r = d <= 32 ? 4 : (d <= 64 ? 8 : (d <= 128 ? 16 : 32));
     int cb = 32;
-    while (cb > 4 && cb / 2 >= dv) cb /= 2;                     // no CTA wider than the head
+    while (cb > 4 && cb / 2 >= columns) cb /= 2;                // no CTA wider than the head
     if (spread) {
         const int sms = sm_count > 0 ? sm_count : 148;
-        while (cb > 8 && n_segments * n_heads * ((dv + cb / 2 - 1) / (cb / 2)) <= sms) cb /= 2;
+        while (cb > 8 && n_segments * n_heads * ((dv + cb / 2 - 1) / (cb / 2)) <= sms) cb /= 2;      // (a column of ones is a CTA too many at worst)
     }
     // asynchronous copies of rows as they lie need every offset and size on 16 bytes; prompt portions only (a step of
     // single tokens has nothing to copy ahead)
@@ -1346,11 +1369,17 @@ IB_EXPORT int ib_state_scan(int mode, const float* rows, int64_t ld, int q_col, 
     chunk = chunk < 1 ? 1 : (chunk > 16 ? 16 : chunk);
     const size_t smem = size_t(n_buf) * chunk * per_token * sizeof(float);
     if (smem > 48 * 1024) return ib::fail(IB_ERR_ARG, "ib_state_scan: a token of %d floats does not fit the staging area", per_token);
-    const dim3 grid{unsigned(n_segments), unsigned(n_heads), unsigned((dv + cb - 1) / cb)};
+    const dim3 grid{unsigned(n_segments), unsigned(n_heads), unsigned((columns + cb - 1) / cb)};
     const int threads = cb * LK;
 #define IB_SCAN(RR, MM)                                                                                                          \
     return launch_scan<RR, MM>(grid, threads, smem, stream, rows, ld, q_col, k_col, v_col, aux, lda, aux_col, state, seg_start, \
-                               seg_slot, raw_out, n_heads, heads_per_qk, d, dv, cb, chunk, write_state, pipelined, bonus, act, scal_col)
+                               seg_slot, raw_out, n_heads, heads_per_qk, d, dv, cb, chunk, write_state, pipelined, bonus, act, scal_col, ones_state, ones_out)
+    if (mode == 5) {
+        if (r == 4) IB_SCAN(4, 5);
+        if (r == 8) IB_SCAN(8, 5);
+        if (r == 16) IB_SCAN(16, 5);
+        IB_SCAN(32, 5);
+    }
     if (mode == 4) {
         if (r == 4) IB_SCAN(4, 4);
         if (r == 8) IB_SCAN(8, 4);

@@ -63,9 +63,11 @@ sum_norm_kernel(const float* __restrict__ x, float alpha, const float* __restric
 // In front of paged attention: projected rows [q (heads x d) | k (kv x d) | v (kv x dv)] from column col0 (the v
 // columns absent where the values are the keys as projected) -> q rows for the attention kernel, k and v into the
 // token's page. One warp per (token, head of q, k or v). q and k heads are divided by their root mean square over d
-// (eps inside the root) and multiplied by a weight [d] that the heads share (wq, wk; null: no norm); then channel
-// pairs (2i, 2i + 1) below n_rot turn by the token's position (tables [positions, n_rot / 2]); q is then multiplied
-// by 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1) (temp_every 0: no temperature). v is stored as projected.
+// (eps inside the root) and multiplied by a weight [d] that the heads share (wq, wk; null: no norm, or with `unit_norm`
+// the division alone); then channel pairs below n_rot turn by the token's position (tables [positions, n_rot / 2]):
+// (2i, 2i + 1), or with `half` (i, i + n_rot / 2); q is then multiplied by 1 + temp_coef * ln(floor((p + 1) / temp_every)
+// + 1) (temp_every 0: no temperature). v is stored as projected. A turn keeps a head's length, so a unit_norm head is
+// the same whether it is divided before or after it.
 template <typename T>
 __global__ void __launch_bounds__(128)
 head_prepare_kernel(const T* __restrict__ rows, int64_t ld, int col0, const float* __restrict__ wq, const float* __restrict__ wk,
@@ -73,10 +75,10 @@ head_prepare_kernel(const T* __restrict__ rows, int64_t ld, int col0, const floa
                     int temp_every, int values_are_keys, const int* __restrict__ positions, const int* __restrict__ token_seg,
                     const int* __restrict__ block_table, int64_t max_blocks, T* __restrict__ q_out, T* __restrict__ k_cache,
                     T* __restrict__ v_cache, int64_t n_tokens, int n_heads, int n_kv, int d, int dv, int page_size,
-                    int write_cache, int64_t n_pages, int* status) {
+                    int write_cache, int64_t n_pages, int* status, int unit_norm, int half_layout) {
     ib::pdl_wait();
     const int lane = threadIdx.x & 31;
-    const int per_token = n_heads + 2 * n_kv;
+    const int per_token = n_heads + (write_cache ? 2 * n_kv : 0);
     const int64_t wi = int64_t(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (wi >= n_tokens * per_token) return;
     const int64_t t = wi / per_token;
@@ -85,7 +87,6 @@ head_prepare_kernel(const T* __restrict__ rows, int64_t ld, int col0, const floa
     const T* r = rows + t * ld + col0;
     const int nq = n_heads * d, nk = n_kv * d;
     const bool is_q = u < n_heads, is_k = !is_q && u < n_heads + n_kv;
-    if (!is_q && !write_cache) return;
     int64_t cache_row = 0;
     if (!is_q) {
         const int page = block_table[int64_t(token_seg[t]) * max_blocks + pos / page_size];
@@ -107,7 +108,7 @@ head_prepare_kernel(const T* __restrict__ rows, int64_t ld, int col0, const floa
     const float* w = is_q ? wq : wk;
     T* dst = is_q ? q_out + t * nq + u * d : k_cache + cache_row * d;
     float f = 1.0f;
-    if (w) {
+    if (w || unit_norm) {
         float ss = 0.0f;
         for (int j = lane; j < d; j += 32) { const float v = ib::to_f32(src[j]); ss = fmaf(v, v, ss); }
         ss = ib::warp_sum(ss);
@@ -116,6 +117,20 @@ head_prepare_kernel(const T* __restrict__ rows, int64_t ld, int col0, const floa
     float mult = 1.0f;
     if (is_q && temp_every > 0) mult = 1.0f + temp_coef * logf(float((pos + 1) / temp_every + 1));
     const int half = n_rot / 2;
+    if (half_layout) {
+        for (int j = lane; j < half; j += 32) {
+            float a = ib::to_f32(src[j]) * f, b = ib::to_f32(src[j + half]) * f;
+            if (w) { a *= w[j]; b *= w[j + half]; }
+            const float c = cos_t[int64_t(pos) * half + j], s = sin_t[int64_t(pos) * half + j];
+            dst[j] = ib::from_f32<T>((a * c - b * s) * mult);
+            dst[j + half] = ib::from_f32<T>((b * c + a * s) * mult);
+        }
+        for (int j = n_rot + lane; j < d; j += 32) {
+            const float a = ib::to_f32(src[j]) * f;
+            dst[j] = ib::from_f32<T>((w ? a * w[j] : a) * mult);
+        }
+        return;
+    }
     for (int p = lane; 2 * p < d; p += 32) {
         const int j = 2 * p;
         float a = ib::to_f32(src[j]) * f, b = j + 1 < d ? ib::to_f32(src[j + 1]) * f : 0.0f;
@@ -130,14 +145,14 @@ head_prepare_kernel(const T* __restrict__ rows, int64_t ld, int col0, const floa
     }
 }
 
-// ctx[t, i] *= sigmoid(rows[t, gate_col + i]) for i < width, in place.
+// ctx[t, i] *= sigmoid(rows[t, gate_col + i / per]) for i < width, in place (per > 1: `per` neighbours share a gate).
 template <typename T>
-__global__ void gate_mul_kernel(T* __restrict__ ctx, const T* __restrict__ rows, int64_t ld, int64_t gate_col, int64_t width, int64_t n) {
+__global__ void gate_mul_kernel(T* __restrict__ ctx, const T* __restrict__ rows, int64_t ld, int64_t gate_col, int64_t width, int64_t per, int64_t n) {
     ib::pdl_wait();
     const int64_t i = int64_t(blockIdx.x) * blockDim.x + threadIdx.x;
     if (i >= n) return;
     const int64_t t = i / width, c = i - t * width;
-    ctx[i] = ib::from_f32<T>(ib::to_f32(ctx[i]) * sigmoid_(ib::to_f32(rows[t * ld + gate_col + c])));
+    ctx[i] = ib::from_f32<T>(ib::to_f32(ctx[i]) * sigmoid_(ib::to_f32(rows[t * ld + gate_col + (per > 1 ? c / per : c)])));
 }
 
 // silu of columns [col0, col0 + width) of float rows, in place.
@@ -197,11 +212,32 @@ double_exp_decay_kernel(const T* __restrict__ rows, int64_t ld, int low_col, int
 
 // One warp per (token, group of `size` channels): out = o / sqrt(mean(o^2) + eps) * w [* act(gate)], o float
 // [tokens, groups * size]; w [groups * size] (null: no weight); the gate's logits are columns gate_col + g size + j
-// of rows `gate` (leading dimension ldg); act: 1 silu, 2 sigmoid, 0 the logits are multipliers as they are.
+// of rows `gate` (leading dimension ldg); act: 1 silu, 2 sigmoid, 0 the logits are multipliers as they are. With
+// `gate_first` the gate multiplies o before the norm instead: out = p / sqrt(mean(p^2) + eps) * w, p = o * act(gate).
+// With `den` [tokens, groups] (how much a group's read-out is worth, and a lower bound at floor_col + g of rows `den_floor`)
+// o is first divided: o' = den_mult * o / (max(|den_mult * den|, floor) + den_eps).
+struct GroupScale {
+    const float* den;
+    const float* den_floor;
+    int64_t ldf;
+    int64_t floor_col;
+    float den_mult, den_eps;
+    __device__ __forceinline__ float at(int64_t t, int g, int n_groups) const {
+        if (!den) return 1.0f;
+        return den_mult / (fmaxf(fabsf(den_mult * den[t * n_groups + g]), den_floor[t * ldf + floor_col + g]) + den_eps);
+    }
+};
+
+template <typename TG>
+__device__ __forceinline__ float gate_value(const TG* gate, int64_t at, int act) {
+    const float z = ib::to_f32(gate[at]);
+    return act == 1 ? silu_(z) : (act == 2 ? sigmoid_(z) : z);
+}
+
 template <typename TG, typename TOut>
 __global__ void group_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, float eps,
                                        const TG* __restrict__ gate, int64_t ldg, int64_t gate_col, int act, TOut* __restrict__ out,
-                                       int64_t n_rows, int n_groups, int size) {
+                                       int64_t n_rows, int n_groups, int size, int gate_first, const GroupScale scale) {
     ib::pdl_wait();
     const int lane = threadIdx.x & 31;
     const int64_t r = int64_t(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -209,17 +245,20 @@ __global__ void group_norm_gate_kernel(const float* __restrict__ o, const float*
     const int64_t t = r / n_groups;
     const int g = int(r - t * n_groups);
     const float* x = o + r * size;
+    const int64_t gate_at = t * ldg + gate_col + int64_t(g) * size;
+    const float pre = scale.at(t, g, n_groups);
     float ss = 0.0f;
-    for (int j = lane; j < size; j += 32) ss = fmaf(x[j], x[j], ss);
+    for (int j = lane; j < size; j += 32) {
+        float v = x[j] * pre;
+        if (gate_first) v *= gate_value(gate, gate_at + j, act);
+        ss = fmaf(v, v, ss);
+    }
     ss = ib::warp_sum(ss);
     const float f = 1.0f / sqrtf(ss / float(size) + eps);
     for (int j = lane; j < size; j += 32) {
-        float y = x[j] * f;
+        float y = x[j] * pre * f;
         if (w) y *= w[int64_t(g) * size + j];
-        if (gate) {
-            const float z = ib::to_f32(gate[t * ldg + gate_col + int64_t(g) * size + j]);
-            y *= act == 1 ? silu_(z) : (act == 2 ? sigmoid_(z) : z);
-        }
+        if (gate) y *= gate_value(gate, gate_at + j, act);
         out[r * size + j] = ib::from_f32<TOut>(y);
     }
 }
@@ -259,24 +298,28 @@ __global__ void relu_sq_vec_kernel(const bf16* __restrict__ rows, int64_t ld, in
 template <typename TG, typename TOut>
 __global__ void __launch_bounds__(256)
 group_norm_gate_wide_kernel(const float* __restrict__ o, const float* __restrict__ w, float eps, const TG* __restrict__ gate,
-                            int64_t ldg, int64_t gate_col, int act, TOut* __restrict__ out, int n_groups, int size) {
+                            int64_t ldg, int64_t gate_col, int act, TOut* __restrict__ out, int n_groups, int size, int gate_first,
+                            const GroupScale scale) {
     ib::pdl_wait();
     __shared__ float red[32];
     const int64_t r = blockIdx.x;
     const int64_t t = r / n_groups;
     const int g = int(r - t * n_groups);
     const float* x = o + r * size;
+    const int64_t gate_at = t * ldg + gate_col + int64_t(g) * size;
+    const float pre = scale.at(t, g, n_groups);
     float ss = 0.0f;
-    for (int j = threadIdx.x; j < size; j += blockDim.x) ss = fmaf(x[j], x[j], ss);
+    for (int j = threadIdx.x; j < size; j += blockDim.x) {
+        float v = x[j] * pre;
+        if (gate_first) v *= gate_value(gate, gate_at + j, act);
+        ss = fmaf(v, v, ss);
+    }
     ss = ib::block_sum(ss, red);
     const float f = 1.0f / sqrtf(ss / float(size) + eps);
     for (int j = threadIdx.x; j < size; j += blockDim.x) {
-        float y = x[j] * f;
+        float y = x[j] * pre * f;
         if (w) y *= w[int64_t(g) * size + j];
-        if (gate) {
-            const float z = ib::to_f32(gate[t * ldg + gate_col + int64_t(g) * size + j]);
-            y *= act == 1 ? silu_(z) : (act == 2 ? sigmoid_(z) : z);
-        }
+        if (gate) y *= gate_value(gate, gate_at + j, act);
         out[r * size + j] = ib::from_f32<TOut>(y);
     }
 }
@@ -335,18 +378,19 @@ IB_EXPORT int ib_head_prepare(const void* rows, int64_t ld, int col0, const floa
                               const float* sin_t, int n_rot, float temp_coef, int temp_every, int values_are_keys,
                               const int* positions, const int* token_seg, const int* block_table, int64_t max_blocks, void* q_out,
                               void* k_cache, void* v_cache, int64_t n_tokens, int n_heads, int n_kv, int d, int dv, int page_size,
-                              int write_cache, int64_t n_pages, int dtype, int* status, cudaStream_t stream) {
+                              int write_cache, int64_t n_pages, int dtype, int* status, cudaStream_t stream, int unit_norm,
+                              int half_layout) {
     if (n_tokens <= 0) return IB_OK;
     if (n_heads <= 0 || n_kv <= 0 || d <= 0 || dv <= 0 || page_size <= 0)
         return ib::fail(IB_ERR_ARG, "ib_head_prepare: bad sizes");
     if (n_rot < 0 || n_rot % 2 || n_rot > d || (n_rot > 0 && (!cos_t || !sin_t)))
         return ib::fail(IB_ERR_ARG, "ib_head_prepare: %d rotated channels of %d need tables and an even count", n_rot, d);
     if (values_are_keys && dv != d) return ib::fail(IB_ERR_ARG, "ib_head_prepare: values that are the keys have the keys' size");
-    const int64_t warps = n_tokens * (n_heads + 2 * n_kv);
+    const int64_t warps = n_tokens * (n_heads + (write_cache ? 2 * n_kv : 0));
 #define IB_HP(TT)                                                                                                                 \
     IB_LAUNCH(head_prepare_kernel<TT>, blocks_for(warps, 4), 128, 0, (const TT*)rows, ld, col0, wq, wk, eps, cos_t, sin_t, n_rot,  \
               temp_coef, temp_every, values_are_keys, positions, token_seg, block_table, max_blocks, (TT*)q_out, (TT*)k_cache,    \
-              (TT*)v_cache, n_tokens, n_heads, n_kv, d, dv, page_size, write_cache, n_pages, status)
+              (TT*)v_cache, n_tokens, n_heads, n_kv, d, dv, page_size, write_cache, n_pages, status, unit_norm, half_layout)
     if (dtype == IB_F32) IB_HP(float);
     else if (dtype == IB_BF16) IB_HP(bf16);
     else return ib::fail(IB_ERR_ARG, "ib_head_prepare: unknown dtype %d", dtype);
@@ -354,12 +398,12 @@ IB_EXPORT int ib_head_prepare(const void* rows, int64_t ld, int col0, const floa
     return ib::check_launch("ib_head_prepare");
 }
 
-IB_EXPORT int ib_gate_mul(void* ctx, const void* rows, int64_t ld, int64_t gate_col, int64_t width, int64_t n_tokens, int dtype,
-                          cudaStream_t stream) {
+IB_EXPORT int ib_gate_mul(void* ctx, const void* rows, int64_t ld, int64_t gate_col, int64_t width, int64_t per, int64_t n_tokens,
+                          int dtype, cudaStream_t stream) {
     const int64_t n = n_tokens * width;
     if (n <= 0) return IB_OK;
-    if (dtype == IB_F32) IB_LAUNCH(gate_mul_kernel<float>, blocks_for(n, 256), 256, 0, (float*)ctx, (const float*)rows, ld, gate_col, width, n);
-    else if (dtype == IB_BF16) IB_LAUNCH(gate_mul_kernel<bf16>, blocks_for(n, 256), 256, 0, (bf16*)ctx, (const bf16*)rows, ld, gate_col, width, n);
+    if (dtype == IB_F32) IB_LAUNCH(gate_mul_kernel<float>, blocks_for(n, 256), 256, 0, (float*)ctx, (const float*)rows, ld, gate_col, width, per, n);
+    else if (dtype == IB_BF16) IB_LAUNCH(gate_mul_kernel<bf16>, blocks_for(n, 256), 256, 0, (bf16*)ctx, (const bf16*)rows, ld, gate_col, width, per, n);
     else return ib::fail(IB_ERR_ARG, "ib_gate_mul: unknown dtype %d", dtype);
     return ib::check_launch("ib_gate_mul");
 }
@@ -418,15 +462,19 @@ IB_EXPORT int ib_double_exp_decay(const void* rows, int64_t ld, int low_col, int
 
 IB_EXPORT int ib_group_norm_gate(const float* o, const float* w, float eps, const void* gate, int64_t ldg, int64_t gate_col,
                                  int gate_dtype, int act, void* out, int out_dtype, int64_t n_tokens, int n_groups, int size,
-                                 cudaStream_t stream) {
+                                 cudaStream_t stream, int gate_first, const float* den, const float* den_floor, int64_t ldf,
+                                 int64_t floor_col, float den_mult, float den_eps) {
     const int64_t rows = n_tokens * n_groups;
     if (rows <= 0 || size <= 0) return IB_OK;
+    if (gate_first && !gate) return ib::fail(IB_ERR_ARG, "ib_group_norm_gate: a gate in front of the norm needs its logits");
+    if (den && !den_floor) return ib::fail(IB_ERR_ARG, "ib_group_norm_gate: a denominator needs its lower bound");
+    const GroupScale scale{den, den_floor, ldf, floor_col, den_mult, den_eps};
     const bool wide = size >= 512;                          // (by the group's size only, never by the number of rows)
     const unsigned grid = wide ? unsigned(rows) : blocks_for(rows, 8);
 #define IB_GN(TG, TO)                                                                                                               \
     do {                                                                                                                            \
-        if (wide) IB_LAUNCH((group_norm_gate_wide_kernel<TG, TO>), grid, 256, 0, o, w, eps, (const TG*)gate, ldg, gate_col, act, (TO*)out, n_groups, size); \
-        else IB_LAUNCH((group_norm_gate_kernel<TG, TO>), grid, 256, 0, o, w, eps, (const TG*)gate, ldg, gate_col, act, (TO*)out, rows, n_groups, size);     \
+        if (wide) IB_LAUNCH((group_norm_gate_wide_kernel<TG, TO>), grid, 256, 0, o, w, eps, (const TG*)gate, ldg, gate_col, act, (TO*)out, n_groups, size, gate_first, scale); \
+        else IB_LAUNCH((group_norm_gate_kernel<TG, TO>), grid, 256, 0, o, w, eps, (const TG*)gate, ldg, gate_col, act, (TO*)out, rows, n_groups, size, gate_first, scale);     \
     } while (0)
     if (!gate || gate_dtype == IB_F32) {
         if (out_dtype == IB_F32) IB_GN(float, float);

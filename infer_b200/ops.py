@@ -596,14 +596,15 @@ def rownorm_store(rows: torch.Tensor, col0: int, wq: Optional[torch.Tensor], wk:
 
 
 def attention_split(q, k_cache, v_cache, block_table, step, n_heads, n_kv, head_dim, v_head_dim, window, scale,
-                    dist_bias=None, sink=None, out=None, single_only=False, keep_first=0, slopes=None, gate=None, gate_col=0):
+                    dist_bias=None, sink=None, out=None, single_only=False, keep_first=0, slopes=None, gate=None, gate_col=0,
+                    gate_per_head=False):
     """Paged attention with keys split over CTAs (chunks of 128 keys aligned to absolute positions, merged in
     ascending order), for tokens that read a few hundred keys each: decoded tokens of a windowed layer. Takes a
     distance bias float32 [L, heads] and a sink float32 [heads]. With ``single_only`` only tokens that are a segment
     of their own are computed (into ``out``, whose other rows stay). ``keep_first``: a windowed query also sees the keys
     at positions below it; ``slopes`` float32 [heads]: slopes[h] * distance is taken off the scaled score. ``gate``
-    (rows in q's dtype, logits of a gate per output channel from column ``gate_col``): the result is multiplied by their
-    sigmoid in the merge."""
+    (rows in q's dtype, logits of a gate per output channel, or with ``gate_per_head`` per head, from column ``gate_col``):
+    the result is multiplied by their sigmoid in the merge."""
     _check(q, "q")
     T = q.shape[0]
     n_pages, ckv, page_size, chd = k_cache.shape
@@ -627,17 +628,19 @@ def attention_split(q, k_cache, v_cache, block_table, step, n_heads, n_kv, head_
         _check(slopes, "slopes", torch.float32, (n_heads,))
     if gate is not None:
         _check(gate, "gate", q.dtype)
-        if gate.shape[0] != T or gate_col < 0 or gate_col + n_heads * v_head_dim > gate.shape[1]:
+        if gate.shape[0] != T or gate_col < 0 or gate_col + n_heads * (1 if gate_per_head else v_head_dim) > gate.shape[1]:
             raise KernelError("the gate columns lie outside the rows")
     n_ws = int(_fn("mix", "ib_attention_split_workspace", [c_int64, c_int, c_int, c_int, c_int], restype=c_int64)(T, n_heads, v_head_dim, visible, keep_first))
     ws = torch.empty(n_ws, dtype=torch.float32, device=q.device)
     f = _fn("mix", "ib_attention_split", [c_void_p] * 4 + [c_int64] + [c_void_p] * 5 + [c_int64] + [c_int] * 6 + [c_float, c_int64,
-                                          c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int64, c_int64])
+                                          c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int64, c_int64,
+                                          c_int])
     _call(f, q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), block_table.shape[1],
           step.token_seg.data_ptr(), step.positions.data_ptr(), step.seg_start.data_ptr() if single_only else None, out.data_ptr(),
           ws.data_ptr(), T, n_heads, n_kv, head_dim, v_head_dim, page_size, int(window or 0), float(scale), n_pages,
           _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0], _ptr(sink), visible, dtype_code(q.dtype),
-          _ptr(step.status), _stream(), keep_first, _ptr(slopes), _ptr(gate), 0 if gate is None else gate.shape[1], int(gate_col))
+          _ptr(step.status), _stream(), keep_first, _ptr(slopes), _ptr(gate), 0 if gate is None else gate.shape[1], int(gate_col),
+          int(bool(gate_per_head)))
     return out
 
 
@@ -764,14 +767,14 @@ def tail_update(rows: torch.Tensor, col0: int, tails: torch.Tensor, seg_start: t
           seg_slot.numel(), _stream())
 
 
-SCAN_ROW_DECAY, SCAN_DELTA_RULE, SCAN_HEAD_DECAY, SCAN_BONUS, SCAN_CHANNEL_DELTA = 0, 1, 2, 3, 4
+SCAN_ROW_DECAY, SCAN_DELTA_RULE, SCAN_HEAD_DECAY, SCAN_BONUS, SCAN_CHANNEL_DELTA, SCAN_STEP = 0, 1, 2, 3, 4, 5
 SCAN_SPREAD_FROM = 8          # segments of more tokens than this spread a head's columns over more CTAs
 
 
 def state_scan(mode: int, rows: torch.Tensor, q_col: int, k_col: int, v_col: int, aux: torch.Tensor, aux_col: int,
                state: torch.Tensor, seg_start: torch.Tensor, seg_slot: torch.Tensor, n_heads: int, heads_per_qk: int,
                dim: int, v_dim: int, write_state: bool = True, max_len: int = 1, bonus: Optional[torch.Tensor] = None,
-               silu: bool = False, scalar_col: int = 0) -> torch.Tensor:
+               silu: bool = False, scalar_col: int = 0, ones_state: Optional[torch.Tensor] = None):
     """A linear recurrence with a float32 matrix state [slots, heads, dim, v_dim], over the tokens of every segment
     in order. SCAN_ROW_DECAY: S <- diag(a) S + k v^T, o = S^T q, with a in ``aux`` columns aux_col + h * dim.
     SCAN_DELTA_RULE: S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q, with ``aux`` columns [g (heads) | beta
@@ -780,7 +783,10 @@ def state_scan(mode: int, rows: torch.Tensor, q_col: int, k_col: int, v_col: int
     [heads] (a constant per head) or [T, ...] with g at column aux_col + h. SCAN_BONUS: o = (S + diag(u) k v^T)^T q, then
     S <- diag(a) S + k v^T, with a as for SCAN_ROW_DECAY and u = ``bonus`` float32 [heads, dim]. SCAN_CHANNEL_DELTA:
     S <- diag(a) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q, with a as for SCAN_ROW_DECAY and ``aux`` columns
-    [beta (heads) | k.q (heads / heads_per_qk)] from ``scalar_col``.
+    [beta (heads) | k.q (heads / heads_per_qk)] from ``scalar_col``. SCAN_STEP: S <- g S + beta k v^T, o = S^T q + skip v,
+    with ``aux`` columns [g (heads) | beta (heads)] from aux_col and skip = ``bonus`` float32 [heads] (None: 0); with
+    ``ones_state`` float32 [slots, heads, dim] one more column whose values are 1, n <- g n + beta k, is kept there and
+    the result is (o, n.q float32 [T, heads]).
     ``silu``: q, k and v are z * sigmoid(z) of what the rows hold (applied while the tokens are staged).
     Returns o float32 [T, heads * v_dim]."""
     _check(rows, "rows", torch.float32)
@@ -811,7 +817,7 @@ def state_scan(mode: int, rows: torch.Tensor, q_col: int, k_col: int, v_col: int
             raise KernelError("a decay per head needs one value per head")
     else:
         need = {SCAN_ROW_DECAY: n_heads * dim, SCAN_BONUS: n_heads * dim, SCAN_DELTA_RULE: 2 * n_heads + n_qk, SCAN_HEAD_DECAY: n_heads,
-                SCAN_CHANNEL_DELTA: n_heads * dim}[mode]
+                SCAN_CHANNEL_DELTA: n_heads * dim, SCAN_STEP: 2 * n_heads}[mode]
         if mode == SCAN_CHANNEL_DELTA and (aux.dim() != 2 or scalar_col < 0 or scalar_col + n_heads + n_qk > aux.shape[1]):
             raise KernelError("the write strengths lie outside their rows")
         if aux.dim() != 2 or aux.shape[0] != T or aux_col + need > aux.shape[1]:
@@ -821,18 +827,28 @@ def state_scan(mode: int, rows: torch.Tensor, q_col: int, k_col: int, v_col: int
         if bonus is None:
             raise KernelError("SCAN_BONUS needs the bonus [heads, dim]")
         _check(bonus, "bonus", torch.float32, (n_heads, dim))
+    elif mode == SCAN_STEP and bonus is not None:
+        _check(bonus, "bonus", torch.float32, (n_heads,))
+    ones_out = None
+    if ones_state is not None:
+        if mode != SCAN_STEP:
+            raise KernelError("a column of ones goes with SCAN_STEP")
+        _check(ones_state, "ones_state", torch.float32)
+        if tuple(ones_state.shape[1:]) != (n_heads, dim):
+            raise KernelError(f"ones_state must be [slots, {n_heads}, {dim}], got {tuple(ones_state.shape)}")
+        ones_out = torch.empty((T, n_heads), dtype=torch.float32, device=rows.device)
     S = seg_slot.numel()
     _check(seg_start, "seg_start", torch.int32, (S + 1,))
     out = torch.empty((T, n_heads * v_dim), dtype=torch.float32, device=rows.device)
     spread = int(max_len) >= SCAN_SPREAD_FROM
     sm_count = torch.cuda.get_device_properties(rows.device).multi_processor_count if spread else 0
     f = _fn("mix", "ib_state_scan", [c_int, c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_int64, c_int, c_void_p, c_void_p,
-                                     c_void_p, c_void_p] + [c_int] * 8 + [c_void_p, c_void_p, c_int, c_int])
+                                     c_void_p, c_void_p] + [c_int] * 8 + [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p])
     _call(f, int(mode), rows.data_ptr(), ld, int(q_col), int(k_col), int(v_col), aux.data_ptr(), lda, int(aux_col),
           state.data_ptr(), seg_start.data_ptr(), seg_slot.data_ptr(), out.data_ptr(), S, n_heads, int(heads_per_qk), dim, v_dim,
-          int(write_state), int(spread), sm_count, _stream(), _ptr(bonus) if mode == SCAN_BONUS else None, int(bool(silu)),
-          int(scalar_col))
-    return out
+          int(write_state), int(spread), sm_count, _stream(), _ptr(bonus) if mode in (SCAN_BONUS, SCAN_STEP) else None, int(bool(silu)),
+          int(scalar_col), _ptr(ones_state), _ptr(ones_out))
+    return out if ones_state is None else (out, ones_out)
 
 
 def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, eps: float, gate: Optional[torch.Tensor], gate_col: int,
@@ -1158,16 +1174,21 @@ def sum_norm(x: torch.Tensor, alpha: float, a: torch.Tensor, sa: float, b: Optio
 def head_prepare(rows: torch.Tensor, col0: int, wq: Optional[torch.Tensor], wk: Optional[torch.Tensor], eps: float,
                  cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], n_rot: int, temp_coef: float, temp_every: int,
                  values_are_keys: bool, step, block_table: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
-                 n_heads: int, n_kv: int, head_dim: int, v_head_dim: int, write_cache: bool = True) -> torch.Tensor:
+                 n_heads: int, n_kv: int, head_dim: int, v_head_dim: int, write_cache: bool = True, unit_norm: bool = False,
+                 layout: str = "pairs", own_kv: bool = True) -> torch.Tensor:
     """Projected rows [.. | q | k | v | ..] (q at column col0; no v columns with ``values_are_keys``: a position's
     value is its key as projected) -> q [T, heads * head_dim]; k and v into the token's page. Every q and k head is
-    divided by its root mean square (eps inside the root) and multiplied by wq / wk [head_dim] (None: no norm); then
-    channel pairs (2i, 2i + 1) below ``n_rot`` turn by the tables cos, sin [positions, n_rot / 2]; then q is multiplied
-    by 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1) (temp_every 0: not)."""
+    divided by its root mean square (eps inside the root) and multiplied by wq / wk [head_dim] (None: no norm, or with
+    ``unit_norm`` the division alone); then channel pairs below ``n_rot`` turn by the tables cos, sin [positions, n_rot / 2]:
+    (2i, 2i + 1) in the "pairs" layout, (i, i + n_rot / 2) in the "half" layout; then q is multiplied
+    by 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1) (temp_every 0: not). Without ``own_kv`` the rows hold q only
+    (the pages are another layer's) and nothing is written to the pages."""
     _check(rows, "rows")
     T, ld = rows.shape
     nq, nk = n_heads * head_dim, n_kv * head_dim
     nv = 0 if values_are_keys else n_kv * v_head_dim
+    if not own_kv:
+        nk, nv, write_cache = 0, 0, False
     if col0 < 0 or ld < col0 + nq + nk + nv:
         raise KernelError("q, k and v lie outside the rows")
     n_pages, ckv, page_size, chd = k_cache.shape
@@ -1185,23 +1206,24 @@ def head_prepare(rows: torch.Tensor, col0: int, wq: Optional[torch.Tensor], wk: 
     q = torch.empty((T, nq), dtype=rows.dtype, device=rows.device)
     f = _fn("post", "ib_head_prepare", [c_void_p, c_int64, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_float, c_int,
                                         c_int, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int64] +
-            [c_int] * 6 + [c_int64, c_int, c_void_p, c_void_p])
+            [c_int] * 6 + [c_int64, c_int, c_void_p, c_void_p, c_int, c_int])
     _call(f, rows.data_ptr(), ld, int(col0), _ptr(wq), _ptr(wk), float(eps), _ptr(cos) if n_rot else None, _ptr(sin) if n_rot else None,
           int(n_rot), float(temp_coef), int(temp_every), int(bool(values_are_keys)), step.positions.data_ptr(), step.token_seg.data_ptr(),
           block_table.data_ptr(), block_table.shape[1], q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), T, n_heads, n_kv,
-          head_dim, v_head_dim, page_size, int(write_cache), n_pages, dtype_code(rows.dtype), _ptr(step.status), _stream())
+          head_dim, v_head_dim, page_size, int(write_cache), n_pages, dtype_code(rows.dtype), _ptr(step.status), _stream(), int(bool(unit_norm)),
+          ROTATION_LAYOUTS[layout])
     return q
 
 
-def gate_mul(ctx: torch.Tensor, rows: torch.Tensor, gate_col: int) -> torch.Tensor:
-    """ctx[t, i] *= sigmoid(rows[t, gate_col + i]), in place; both in one storage dtype."""
+def gate_mul(ctx: torch.Tensor, rows: torch.Tensor, gate_col: int, per: int = 1) -> torch.Tensor:
+    """ctx[t, i] *= sigmoid(rows[t, gate_col + i // per]), in place; both in one storage dtype."""
     _check(ctx, "ctx")
     _check(rows, "rows", ctx.dtype)
     T, W = ctx.shape
-    if rows.shape[0] != T or gate_col < 0 or gate_col + W > rows.shape[1]:
+    if rows.shape[0] != T or gate_col < 0 or per < 1 or gate_col + -(-W // per) > rows.shape[1]:
         raise KernelError("the gate columns lie outside the rows")
-    f = _fn("post", "ib_gate_mul", [c_void_p, c_void_p, c_int64, c_int64, c_int64, c_int64, c_int, c_void_p])
-    _call(f, ctx.data_ptr(), rows.data_ptr(), rows.shape[1], int(gate_col), W, T, dtype_code(ctx.dtype), _stream())
+    f = _fn("post", "ib_gate_mul", [c_void_p, c_void_p, c_int64, c_int64, c_int64, c_int64, c_int64, c_int, c_void_p])
+    _call(f, ctx.data_ptr(), rows.data_ptr(), rows.shape[1], int(gate_col), W, int(per), T, dtype_code(ctx.dtype), _stream())
     return ctx
 
 
@@ -1257,10 +1279,14 @@ GATE_ACTS = {None: 0, "silu": 1, "sigmoid": 2}
 
 
 def group_norm_gate(o: torch.Tensor, weight: Optional[torch.Tensor], eps: float, gate: Optional[torch.Tensor], gate_col: int,
-                    act: Optional[str], n_groups: int, size: int, out_dtype: torch.dtype) -> torch.Tensor:
+                    act: Optional[str], n_groups: int, size: int, out_dtype: torch.dtype, gate_first: bool = False,
+                    den: Optional[torch.Tensor] = None, den_floor: Optional[torch.Tensor] = None, floor_col: int = 0,
+                    den_mult: float = 1.0, den_eps: float = 0.0) -> torch.Tensor:
     """Per (token, group of ``size`` channels): o / sqrt(mean(o^2) + eps) * weight [groups * size] (None: no weight),
     times act(gate logits) (columns gate_col + g * size of rows ``gate``, float32 or bfloat16; ``act`` "silu", "sigmoid"
-    or None for multipliers as they are) if given. o float32 [T, groups * size]."""
+    or None for multipliers as they are) if given. o float32 [T, groups * size]. ``gate_first``: the gate multiplies o
+    before the norm instead. ``den`` float32 [T, groups] with ``den_floor`` (float32 rows, a lower bound per group from
+    ``floor_col``): o is first replaced by den_mult * o / (max(|den_mult * den|, floor) + den_eps)."""
     _check(o, "o", torch.float32)
     T = o.shape[0]
     _check(o, "o", None, (T, n_groups * size))
@@ -1272,11 +1298,17 @@ def group_norm_gate(o: torch.Tensor, weight: Optional[torch.Tensor], eps: float,
         ldg = gate.shape[1]
         if gate.shape[0] != T or gate_col < 0 or gate_col + n_groups * size > ldg:
             raise KernelError("the gate columns lie outside the rows")
+    if den is not None:
+        _check(den, "den", torch.float32, (T, n_groups))
+        _check(den_floor, "den_floor", torch.float32)
+        if den_floor.shape[0] != T or floor_col < 0 or floor_col + n_groups > den_floor.shape[1]:
+            raise KernelError("the lower bounds lie outside their rows")
     out = torch.empty((T, n_groups * size), dtype=out_dtype, device=o.device)
     f = _fn("post", "ib_group_norm_gate", [c_void_p, c_void_p, c_float, c_void_p, c_int64, c_int64, c_int, c_int, c_void_p, c_int, c_int64,
-                                           c_int, c_int, c_void_p])
+                                           c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int64, c_int64, c_float, c_float])
     _call(f, o.data_ptr(), _ptr(weight), float(eps), _ptr(gate), ldg, int(gate_col), dtype_code(gate.dtype) if gate is not None else 0,
-          GATE_ACTS[act], out.data_ptr(), dtype_code(out_dtype), T, int(n_groups), int(size), _stream())
+          GATE_ACTS[act], out.data_ptr(), dtype_code(out_dtype), T, int(n_groups), int(size), _stream(), int(bool(gate_first)), _ptr(den),
+          _ptr(den_floor), 0 if den_floor is None else den_floor.shape[1], int(floor_col), float(den_mult), float(den_eps))
     return out
 
 
@@ -1451,4 +1483,80 @@ def talk_attention_split(q: torch.Tensor, q_col: int, k_cache: torch.Tensor, v_c
           step.seg_start.data_ptr() if single_only else None, out.data_ptr(), ws.data_ptr(), T, n_heads, n_kv, head_dim, v_head_dim,
           page_size, int(window or 0), int(chunk or 0), n_chunks, float(scale), float(cap or 0.0), _ptr(talk), n_pages, _ptr(step.status),
           _stream())
+    return out
+
+
+# ----------------------------------------------------------------------------- scaled sums, state space layers, matrix memories
+
+def scaled_sum_norm(x: torch.Tensor, a: Optional[torch.Tensor], wa: Optional[torch.Tensor], b: Optional[torch.Tensor],
+                    wb: Optional[torch.Tensor], weight: torch.Tensor, eps: float, out_dtype: torch.dtype,
+                    rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """y = x + wa * a + wb * b per row (float32 [T, W]; a and b may be absent; wa, wb float32 [W]), kept in x; returns
+    y / sqrt(mean(y^2) + eps) * weight in ``out_dtype``. ``rows`` (int32) picks and orders rows (x stays as it is then)."""
+    _check(x, "x", torch.float32)
+    T, W = x.shape
+    for name, t, w in (("a", a, wa), ("b", b, wb)):
+        if t is not None:
+            _check(t, name, torch.float32, (T, W))
+            _check(w, "w" + name, torch.float32, (W,))
+    _check(weight, "weight", torch.float32, (W,))
+    if rows is not None:
+        _check(rows, "rows", torch.int32)
+    n = T if rows is None else rows.numel()
+    out = torch.empty((n, W), dtype=out_dtype, device=x.device)
+    f = _fn("memory", "ib_scaled_sum_norm", [c_void_p] * 6 + [c_float, c_void_p, c_int, c_void_p, c_int, c_int64, c_int64, c_void_p])
+    _call(f, x.data_ptr(), _ptr(a), _ptr(wa), _ptr(b), _ptr(wb), weight.data_ptr(), float(eps), _ptr(rows), int(rows is None),
+          out.data_ptr(), dtype_code(out_dtype), n, W, _stream())
+    return out
+
+
+def filter_prepare(rows: torch.Tensor, col0: int, filt_w: torch.Tensor, filt_b: torch.Tensor, tails: Optional[torch.Tensor], dt_col: int,
+                   dt_bias: torch.Tensor, a_log: torch.Tensor, step, inline_tail: bool = False):
+    """What a state space layer's recurrence reads, from float32 projected rows: columns [col0, col0 + C) each through a
+    causal filter (``filt_w`` float32 [taps, C], ``filt_b`` [C], ``tails`` float32 [slots, taps - 1, C]: the inputs before the
+    step) and silu; per head, from column dt_col, dt = softplus(raw + dt_bias) and g = exp(-exp(a_log) dt). Returns (float32
+    rows [C | up to a multiple of 4 | g (heads) | dt (heads)], first column of g). ``inline_tail`` (steps of one token per
+    request only): the kernel also moves the tails (no ``tail_update``)."""
+    _check(rows, "rows", torch.float32)
+    T, ld = rows.shape
+    _check(filt_w, "filt_w", torch.float32)
+    taps, C = filt_w.shape
+    _check(filt_b, "filt_b", torch.float32, (C,))
+    H = a_log.numel()
+    _check(a_log, "a_log", torch.float32, (H,))
+    _check(dt_bias, "dt_bias", torch.float32, (H,))
+    if col0 < 0 or col0 + C > ld or dt_col < 0 or dt_col + H > ld:
+        raise KernelError("filter_prepare: columns lie outside the rows")
+    if taps > 1:
+        _check(tails, "tails", torch.float32)
+        if tuple(tails.shape[1:]) != (taps - 1, C):
+            raise KernelError(f"tails must be [slots, {taps - 1}, {C}], got {tuple(tails.shape)}")
+    g_col = -(-C // 4) * 4
+    out = torch.empty((T, -(-(g_col + 2 * H) // 4) * 4), dtype=torch.float32, device=rows.device)
+    f = _fn("memory", "ib_filter_prepare", [c_void_p, c_int64, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p,
+                                            c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int64, c_void_p])
+    _call(f, rows.data_ptr(), ld, int(col0), C, filt_w.data_ptr(), filt_b.data_ptr(), taps, _ptr(tails) if taps > 1 else None,
+          int(bool(inline_tail)), int(dt_col), dt_bias.data_ptr(), a_log.data_ptr(), H, step.token_seg.data_ptr(), step.seg_start.data_ptr(),
+          step.seg_slot.data_ptr(), out.data_ptr(), out.shape[1], T, _stream())
+    return out, g_col
+
+
+def memory_gates(rows: torch.Tensor, i_col: int, f_col: int, i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float, state: torch.Tensor,
+                 step, write_state: bool = True) -> torch.Tensor:
+    """Gates of a matrix memory over the tokens of every segment in order, from float32 projected rows: with
+    i = cap tanh((raw_i + i_bias) / cap) and f = log sigmoid(cap tanh((raw_f + f_bias) / cap)) per head, m <- max(f + m, i)
+    (kept in ``state`` float32 [slots, heads]). Returns float32 [T, exp(f + m_before - m) | exp(i - m) | exp(-m)], heads each."""
+    _check(rows, "rows", torch.float32)
+    T, ld = rows.shape
+    H = i_bias.numel()
+    _check(i_bias, "i_bias", torch.float32, (H,))
+    _check(f_bias, "f_bias", torch.float32, (H,))
+    _check(state, "state", torch.float32, (state.shape[0], H))
+    if min(i_col, f_col) < 0 or max(i_col, f_col) + H > ld:
+        raise KernelError("memory_gates: columns lie outside the rows")
+    out = torch.empty((T, 3 * H), dtype=torch.float32, device=rows.device)
+    f = _fn("memory", "ib_memory_gates", [c_void_p, c_int64, c_int, c_int, c_void_p, c_void_p, c_float] + [c_void_p] * 4 +
+            [c_int64, c_int, c_int, c_int, c_void_p])
+    _call(f, rows.data_ptr(), ld, int(i_col), int(f_col), i_bias.data_ptr(), f_bias.data_ptr(), float(cap), state.data_ptr(),
+          step.seg_start.data_ptr(), step.seg_slot.data_ptr(), out.data_ptr(), 3 * H, step.seg_slot.numel(), H, int(write_state), _stream())
     return out

@@ -30,15 +30,22 @@ Options beyond that, each a key of the part's spec (absent = off):
 A third group of options goes through one kernel that normalises per head, rotates, applies the temperature and
 fills the pages (``head_prepare``), then through the attention kernels that take a slope and kept first keys:
 
+``qk_unit_norm_eps``   every q head and every k head is divided by its root mean square over head_dim, without a weight;
+                       with a rotation it is all one whether before or after it (a turn keeps a head's length)
 ``qk_head_norm_eps``   EVERY q head and every k head is divided by its own root mean square over head_dim and
                        multiplied by a weight [head_dim] that the heads share (roles q_norm, k_norm), before any
-                       rotation; ``position`` may then be "rotary_interpolated" in the pairs layout (or none)
+                       rotation; ``position`` may then be "rotary_interpolated" in either layout (or none)
 ``query_temperature``  {"coef": c, "every": n}: q at position p is multiplied by 1 + c ln(floor((p + 1) / n) + 1)
 ``distance_slopes``    a number per head: slope_h * (i - j) is taken off the scaled score of query i and key j
 ``keep_first``         with a window: query i also sees every key j < keep_first (at its true position)
 ``values_are_keys``    there is no v matrix: a position's value is its key as projected, before norm and rotation
 ``channel_gate``       the joined heads are multiplied, channel by channel, by sigmoid(x Wg^T) (role gate,
                        [heads * v_head_dim, hidden]) before the output product; Wg rides in the q/k/v product
+``head_gate``          as above, beside the options of this group
+``own_kv``             False: no k and v matrices; the layer reads the keys and values that another layer of the same sizes
+                       and rotation left in its cache (the run order names that cache), with its own queries and mask
+``cache_window``, ``cache_keep_first``   what the pages must hold where several layers read them (default: the layer's own
+                       window and kept first keys)
 ``sink``               as above
 
 A fourth group goes through kernels that work on all heads of a (query, key) pair at once:
@@ -126,7 +133,8 @@ class Attention(Mixer):
         self.value_norm_eps = spec.get("value_norm_eps")
         self.head_gate = bool(spec.get("head_gate", False))
         # anything beyond rotate-and-store goes through the prepare kernel (filter, pair rotation, value norm)
-        if getattr(self.position, "layout", "half") == "half" and self.position is not None and self.head_dim % 2:
+        if self.position is not None and getattr(self.position, "layout", "half") == "half" and not hasattr(self.position, "rotary_dims") \
+                and self.head_dim % 2:
             raise ValueError(f"half-split rotation needs an even head_dim, got {self.head_dim}")
         self.prepared = (self.taps > 0 or self.value_norm_eps is not None or self.v_dim != self.head_dim or self.head_gate
                          or getattr(self.position, "layout", "half") == "pairs")
@@ -136,9 +144,12 @@ class Attention(Mixer):
         self.slopes = [float(v) for v in spec["distance_slopes"]] if spec.get("distance_slopes") is not None else None
         self.keep_first = int(spec.get("keep_first") or 0)
         self.values_are_keys = bool(spec.get("values_are_keys", False))
+        self.unit_norm_eps = spec.get("qk_unit_norm_eps")
+        self.own_kv = bool(spec.get("own_kv", True))
+        self.cache_window, self.cache_keep = spec.get("cache_window", self.window), int(spec.get("cache_keep_first", self.keep_first) or 0)
         self.channel_gate = bool(spec.get("channel_gate", False))
         self.per_head = (self.head_norm_eps is not None or self.q_temp is not None or self.slopes is not None or self.keep_first > 0
-                         or self.values_are_keys or self.channel_gate)
+                         or self.values_are_keys or self.channel_gate or self.unit_norm_eps is not None or not self.own_kv)
         if self.per_head:
             self._check_per_head(spec)
         self.cap = float(spec.get("score_cap") or 0.0)
@@ -174,19 +185,33 @@ class Attention(Mixer):
             self.biased = False
         self.q_norm_w = self.k_norm_w = self.bias_table = self.bias_by_head = self.sink_w = self.slopes_w = None
         self.n_qkv = (self.n_heads + self.n_kv) * self.head_dim + (0 if self.values_are_keys else self.n_kv * self.v_dim)
+        if not self.own_kv:
+            self.n_qkv = self.n_heads * self.head_dim
         self.qkv: Optional[Linear] = None
         self.o: Optional[Linear] = None
         self.filter_w = None
 
     def _check_per_head(self, spec):
-        if self.taps > 0 or self.value_norm_eps is not None or self.head_gate or self.qkv_bias or spec.get("qk_row_norm_eps") is not None \
+        if self.taps > 0 or self.value_norm_eps is not None or self.qkv_bias or spec.get("qk_row_norm_eps") is not None \
                 or spec.get("distance_bias") is not None:
-            raise ValueError("per-head norms, temperature, slopes, kept first keys, keys as values and channel gates do not combine "
-                             "with filters, value norm, head gates, biases, row norms or a distance table")
-        if self.head_norm_eps is not None and float(self.head_norm_eps) <= 0:
-            raise ValueError("qk_head_norm_eps must be positive")
-        if self.position is not None and (getattr(self.position, "layout", None) != "pairs" or self.position.rotary_tables is None):
-            raise ValueError("this attention rotates channel pairs from tables (position kind 'rotary_interpolated' or 'rotary_pairs' in the pairs layout)")
+            raise ValueError("per-head norms, temperature, slopes, kept first keys, keys as values, gates and shared pages do not combine "
+                             "with filters, value norm, biases, row norms or a distance table")
+        if self.head_gate and self.channel_gate:
+            raise ValueError("a gate per head or per channel, not both")
+        for eps in (self.head_norm_eps, self.unit_norm_eps):
+            if eps is not None and float(eps) <= 0:
+                raise ValueError("qk_head_norm_eps and qk_unit_norm_eps must be positive")
+        if self.head_norm_eps is not None and self.unit_norm_eps is not None:
+            raise ValueError("q and k heads are normalised with a weight or without one, not both")
+        if self.position is not None and (getattr(self.position, "layout", None) not in ops.ROTATION_LAYOUTS or not hasattr(self.position, "rotary_dims")):
+            raise ValueError("this attention rotates channel pairs from tables (position kind 'rotary_interpolated' or 'rotary_pairs')")
+        if self.unit_norm_eps is not None and getattr(self.position, "scaling", None):
+            raise ValueError("unit-norm heads go with a rotation that keeps a head's length")
+        if self.cache_window is None and self.window is not None:
+            self.cache_keep = 0                              # every position stays
+        elif self.window is None and self.cache_window is not None or \
+                (self.window is not None and (self.cache_window < self.window or self.cache_keep < self.keep_first)):
+            raise ValueError("cache_window and cache_keep_first must cover the layer's own window and kept keys")
         if self.q_temp is not None and (int(self.q_temp.get("every", 0)) <= 0 or "coef" not in self.q_temp):
             raise ValueError("query_temperature needs 'coef' and a positive 'every'")
         if self.slopes is not None and len(self.slopes) != self.n_heads:
@@ -212,7 +237,9 @@ class Attention(Mixer):
         vd = int(spec.get("v_head_dim") or hd)
         n = _names(spec)
         shapes = {n["q"]: (nh * hd, H), n["k"]: (nkv * hd, H), n["v"]: (nkv * vd, H), n["o"]: (H, nh * vd)}
-        if spec.get("values_are_keys", False):
+        if not spec.get("own_kv", True):
+            del shapes[n["k"]], shapes[n["v"]]
+        elif spec.get("values_are_keys", False):
             del shapes[n["v"]]
         if spec.get("channel_gate", False):
             shapes[n["gate"]] = (nh * vd, H)
@@ -256,7 +283,9 @@ class Attention(Mixer):
 
     def load(self, params):
         n = _names(self.spec)
-        mats = [params[n["q"]], params[n["k"]]] + ([] if self.values_are_keys else [params[n["v"]]])
+        mats = [params[n["q"]]]
+        if self.own_kv:
+            mats += [params[n["k"]]] + ([] if self.values_are_keys else [params[n["v"]]])
         if self.head_gate or self.channel_gate:
             mats.append(params[n["gate"]])
         w = torch.cat(mats, dim=0)
@@ -291,8 +320,8 @@ class Attention(Mixer):
                 .to(device=self.rt.device, dtype=torch.float32).t().contiguous()
 
     def cache_need(self):
-        pages = PagedKVNeed(self.n_kv, self.head_dim, self.window, None if self.v_dim == self.head_dim else self.v_dim,
-                            keep_first=self.keep_first if self.window is not None else 0, chunk=self.chunk)
+        pages = PagedKVNeed(self.n_kv, self.head_dim, self.cache_window, None if self.v_dim == self.head_dim else self.v_dim,
+                            keep_first=self.cache_keep if self.cache_window is not None else 0, chunk=self.chunk)
         if self.taps > 1:
             # the last taps - 1 projected rows of the request, in the compute dtype (copies, not sums)
             return CompositeNeed({"pages": pages, "tails": StateNeed({"qkv": ((self.taps - 1, self.n_qkv), None)})})
@@ -337,25 +366,29 @@ class Attention(Mixer):
         return self._project_out(ctx, residual)
 
     def _forward_per_head(self, qkv, col0, step, cache, residual, write_cache):
-        """Per-head norms, pair rotation, the queries' temperature and the cache write in one kernel; attention whose
+        """Per-head norms, rotation, the queries' temperature and the cache write in one kernel; attention whose
         scores lose a slope times the distance, whose window keeps the first keys and whose denominator takes the sink;
-        the gate per channel. The part's columns [q | k | (v) | gate] start at ``col0`` of the rows ``qkv``."""
+        the gate per channel or head. The part's columns [q | (k) | (v) | gate] start at ``col0`` of the rows ``qkv``."""
         table = step.block_tables[cache.group]
         cos = sin = None
         n_rot = 0
         if self.position is not None:
             cos, sin = self.position.rotary_tables(self.rt.max_seq_len)
             n_rot = self.position.rotary_dims
+        if write_cache and not self.own_kv:
+            raise ValueError("an attention layer without keys and values of its own cannot write a cache")
+        layout = self.position.layout if self.position is not None else "pairs"
         coef, every = (float(self.q_temp["coef"]), int(self.q_temp["every"])) if self.q_temp is not None else (0.0, 0)
-        q = ops.head_prepare(qkv, col0, self.q_norm_w, self.k_norm_w, float(self.head_norm_eps or 0.0), cos, sin, n_rot, coef, every,
-                             self.values_are_keys, step, table, cache.k, cache.v, self.n_heads, self.n_kv, self.head_dim, self.v_dim,
-                             write_cache)
+        q = ops.head_prepare(qkv, col0, self.q_norm_w, self.k_norm_w, float(self.head_norm_eps or self.unit_norm_eps or 0.0), cos, sin, n_rot,
+                             coef, every, self.values_are_keys, step, table, cache.k, cache.v, self.n_heads, self.n_kv, self.head_dim,
+                             self.v_dim, write_cache, self.unit_norm_eps is not None, layout, self.own_kv)
         ctx = None
         if self.rt.fast("attention") and step.max_q_len <= 1 and self.n_heads // self.n_kv <= ops.ATTENTION_SPLIT_GROUP_MAX:
             # single tokens only: the kernel that merges a token's key chunks also applies the gate
             ctx = ops.attention_split(q, cache.k, cache.v, table, step, self.n_heads, self.n_kv, self.head_dim, self.v_dim, self.window,
                                       self.scale, None, self.sink_w, keep_first=self.keep_first, slopes=self.slopes_w,
-                                      gate=qkv if self.channel_gate else None, gate_col=col0 + self.n_qkv)
+                                      gate=qkv if self.channel_gate or self.head_gate else None, gate_col=col0 + self.n_qkv,
+                                      gate_per_head=self.head_gate)
             return self._project_out(ctx, residual)
         if self.rt.fast("attention"):
             ctx = ops.attention_window(q, cache.k, cache.v, table, step, self.n_heads, self.n_kv, self.head_dim, self.v_dim,
@@ -364,8 +397,8 @@ class Attention(Mixer):
             ctx = ops.attention_plain(q, cache.k, cache.v, table, step.token_seg, step.positions, self.n_heads, self.n_kv,
                                       self.head_dim, self.window, self.scale, step.status, self.v_dim, None, self.sink_w,
                                       keep_first=self.keep_first, slopes=self.slopes_w)
-        if self.channel_gate:
-            ops.gate_mul(ctx, qkv, col0 + self.n_qkv)
+        if self.channel_gate or self.head_gate:
+            ops.gate_mul(ctx, qkv, col0 + self.n_qkv, self.v_dim if self.head_gate else 1)
         return self._project_out(ctx, residual)
 
     def _forward_all_heads(self, qkv, col0, step, cache, residual, write_cache):

@@ -22,7 +22,12 @@ constants), which also leaves h in the compute dtype for the next sublayer's fir
 
 "hyper_prenorm": prenorm over several residual streams (parts/streams.py). Slots: mixer_norm, mixer_link, mixer,
 feed_forward_norm, feed_forward_link, feed_forward (the last three may be absent together); the links are of family
-"connection". h is a ``StreamRows``; each sublayer's result stays pending there for the kernel that reads next."""
+"connection". h is a ``StreamRows``; each sublayer's result stays pending there for the kernel that reads next.
+
+"parallel_scaled": ONE norm, whose rows n = norm(h) both sublayers read, and a stored factor per channel on what each
+returns: h += s1 * mixer(n) + s2 * feed_forward(n); the feed-forward and its factors may be absent. Slots: norm, mixer,
+mixer_scale, feed_forward, feed_forward_scale (the scales of family "connection"). h is a ``PendingRows``
+(parts/streams.py): the sum is the next norm's kernel."""
 from __future__ import annotations
 
 import os
@@ -264,4 +269,43 @@ class HyperPreNormBlock(Block):
             n = h.read(self.feed_forward_link, self.feed_forward_norm, dtype)
             y = self.feed_forward.forward(n, None) if side is None else self.feed_forward.forward(n, None, side)
             h.write(self.feed_forward_link, y)
+        return h
+
+
+@register_block("parallel_scaled")
+class ParallelScaledBlock(Block):
+    def __init__(self, norm, mixer, mixer_scale, feed_forward=None, feed_forward_scale=None):
+        parts = {"norm": norm, "mixer": mixer, "mixer_scale": mixer_scale}
+        if feed_forward is not None:
+            if feed_forward_scale is None:
+                raise ValueError("a feed-forward in a parallel_scaled block needs its scale")
+            parts.update(feed_forward=feed_forward, feed_forward_scale=feed_forward_scale)
+        super().__init__(**parts)
+        self.feed_forward = feed_forward
+        if not getattr(norm, "fusable", False):
+            raise ValueError("a parallel_scaled block needs a norm of the (weight, eps) root-mean-square kind")
+
+    def forward(self, h, step, cache, write_cache=True):
+        dtype = self.mixer.rt.dtype
+        n = h.read(self.norm, dtype)
+        # In a decode step every kernel is a few microseconds of latency: the feed-forward's chain runs beside the mixer's
+        # (and a router beside the experts' first product), on side streams that join before the sum.
+        side = _side_streams(h.device) if (PARALLEL_BRANCHES and step.decode_only and dtype != torch.float32
+                                           and self.feed_forward is not None) else None
+        if side is None:
+            h.write(self.mixer_scale, self.mixer.forward(n, step, cache, None, write_cache))
+            if self.feed_forward is not None:
+                h.write(self.feed_forward_scale, self.feed_forward.forward(n, None))
+            return h
+        main = torch.cuda.current_stream(h.device)
+        fork, done = torch.cuda.Event(), torch.cuda.Event()
+        fork.record(main)
+        side[0].wait_event(fork)
+        with torch.cuda.stream(side[0]):
+            y = self.feed_forward.forward(n, None, side[1]) if getattr(self.feed_forward, "takes_side_stream", False) \
+                else self.feed_forward.forward(n, None)
+            done.record(side[0])
+        h.write(self.mixer_scale, self.mixer.forward(n, step, cache, None, write_cache))
+        main.wait_event(done)
+        h.write(self.feed_forward_scale, y)
         return h

@@ -123,7 +123,7 @@ def interpolated_frequencies(rotary_dims: int, theta: float, scaling):
 class RotaryInterpolated(PositionEncoding):
     """A rotation over the first ``rotary_dims`` channels of what it is applied to, in either layout ("pairs":
     channel 2i with 2i + 1; "half": channel i with i + rotary_dims / 2), with optionally interpolated frequencies
-    (``scaling``, see interpolated_frequencies). Angles, cosines and sines are computed in float64 on the host and
+    (``scaling``, see interpolated_frequencies), or with every frequency divided by ``linear_factor``. Angles, cosines and sines are computed in float64 on the host and
     rounded once; the magnitude is part of the tables, so the kernels that apply them know nothing of the scaling."""
 
     def __init__(self, spec: PartSpec, runtime):
@@ -133,14 +133,17 @@ class RotaryInterpolated(PositionEncoding):
         self.head_dim = int(spec.get("head_dim") or self.rotary_dims)
         self.layout = str(spec.get("layout", "half"))
         self.scaling = dict(spec["scaling"]) if spec.get("scaling") else None
+        self.linear_factor = float(spec.get("linear_factor") or 1.0)
         self.max_positions = int(spec["max_positions"])
         if self.layout not in ("pairs", "half"):
             raise ValueError(f"a rotation's layout is 'pairs' or 'half', not {self.layout!r}")
         if self.rotary_dims <= 0 or self.rotary_dims % 2 or self.rotary_dims > self.head_dim:
             raise ValueError(f"rotary_interpolated needs an even number of rotated channels within the head, got "
                              f"{self.rotary_dims} of {self.head_dim}")
-        if self.theta <= 1:
-            raise ValueError("rotary_interpolated needs a theta above 1")
+        if self.theta <= 0 or (self.theta <= 1 and self.scaling is not None):
+            raise ValueError("rotary_interpolated needs a positive theta (above 1 where frequencies are interpolated)")
+        if self.linear_factor <= 0:
+            raise ValueError("rotary_interpolated needs a positive linear_factor")
         if self.scaling is not None:
             for k in ("factor", "original", "fast", "slow"):
                 if k not in self.scaling or float(self.scaling[k]) <= 0:
@@ -149,11 +152,11 @@ class RotaryInterpolated(PositionEncoding):
     def rotary_tables(self, n_positions: int = None):
         n = min(self.max_positions, n_positions or self.max_positions)
         sc = tuple(sorted(self.scaling.items())) if self.scaling else None
-        cache_key = ("interpolated", self.rotary_dims, self.theta, sc, n, str(self.rt.device))
+        cache_key = ("interpolated", self.rotary_dims, self.theta, sc, self.linear_factor, n, str(self.rt.device))
         t = _SHARED_TABLES.get(cache_key)
         if t is None:
             freq, mag = interpolated_frequencies(self.rotary_dims, self.theta, self.scaling)
-            angle = torch.arange(n, dtype=torch.float64)[:, None] * freq[None, :]
+            angle = torch.arange(n, dtype=torch.float64)[:, None] * (freq / self.linear_factor)[None, :]
             t = ((torch.cos(angle) * mag).to(torch.float32).to(self.rt.device).contiguous(),
                  (torch.sin(angle) * mag).to(torch.float32).to(self.rt.device).contiguous())
             _SHARED_TABLES[cache_key] = t

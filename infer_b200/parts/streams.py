@@ -101,3 +101,76 @@ class CopiedStream(Stream):
 
     def close(self, h, norm, rows):
         return h.close(norm, rows, self.rt.dtype)
+
+
+# ----------------------------------------------------------------------------- one row per token, results pending
+
+class PendingRows:
+    """The residual rows of a step's tokens, float32 [T, width], and what the last layer's sublayers returned, each with the
+    factor per channel it enters through: whoever reads next takes it in, in the same kernel as its norm."""
+
+    def __init__(self, rows: torch.Tensor):
+        self.rows = rows
+        self.pending = []                      # [(y float32 [T, width], factors float32 [width])], at most two
+
+    @property
+    def device(self):
+        return self.rows.device
+
+    def _terms(self):
+        flat = [t for pair in self.pending for t in pair]
+        return flat + [None] * (4 - len(flat))
+
+    def read(self, norm, dtype: torch.dtype) -> torch.Tensor:
+        """Takes in what is pending; returns norm(rows) in ``dtype``."""
+        out = ops.scaled_sum_norm(self.rows, *self._terms(), norm.weight, norm.eps, dtype)
+        self.pending = []
+        return out
+
+    def write(self, link: "ChannelScale", y: torch.Tensor) -> None:
+        assert len(self.pending) < 2, "two results are pending already"
+        self.pending.append((y, link.weight))
+
+    def total(self) -> torch.Tensor:
+        """float32 [T, width]: the rows with what is pending taken in (a copy; the rows stay as they are)."""
+        rows = self.rows.clone()
+        for y, w in self.pending:
+            rows += y * w
+        return rows
+
+    def close(self, norm, rows: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
+        return ops.scaled_sum_norm(self.rows, *self._terms(), norm.weight, norm.eps, dtype, rows=rows)
+
+
+@register_connection("channel_scale")
+class ChannelScale(Connection):
+    """A sublayer's result enters the residual stream times a stored factor per channel."""
+
+    def __init__(self, spec: PartSpec, runtime):
+        super().__init__(spec, runtime)
+        self.size = int(spec["size"])
+        if self.size <= 0:
+            raise ValueError("channel_scale needs a positive size")
+        self.weight = None
+
+    @classmethod
+    def param_shapes(cls, spec):
+        return {str(spec.get("weight_name", "scale")): (int(spec["size"]),)}
+
+    @classmethod
+    def init_params(cls, spec, name, shape, gen):
+        return 1.0 + 0.2 * torch.randn(shape, generator=gen, dtype=torch.float32, device=gen.device)
+
+    def load(self, params):
+        self.weight = params[str(self.spec.get("weight_name", "scale"))].to(device=self.rt.device, dtype=torch.float32).contiguous()
+
+
+@register_stream("pending_sum")
+class PendingSum(Stream):
+    """One row per token that starts as the embedding's; a layer's results stay pending until the next norm."""
+
+    def open(self, rows):
+        return PendingRows(rows)
+
+    def close(self, h, norm, rows):
+        return h.close(norm, rows, self.rt.dtype)
