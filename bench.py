@@ -7,6 +7,7 @@ random weights on one B200.
     python bench.py --design pefazen [--sizes 1.5b|7b] [--layers L]     (beside Fozerax, the closest design, and Qwen2)
     python bench.py --design biravik [--sizes 1.5b|7b] [--layers L]     (beside Fozerax, the closest design, and Qwen2)
     python bench.py --design notirax [--sizes 1.5b|7b] [--layers L]     (beside Fozerax, the closest design, and Qwen2)
+    python bench.py --design bolelix [--sizes 1.5b|7b] [--layers L]     (beside Biravik, the closest design, and Qwen2)
 
 Prints ONE JSON line. "value" is decoded tokens per second of the step function, timed on the device with CUDA
 events around K decode steps of a batch of 8 requests whose 2,048-token contexts already lie in the paged cache
@@ -39,9 +40,9 @@ SIZES = {"1.5b": _preset("qwen2.5-1.5b"), "7b": _preset("qwen2.5-7b"), "14b": _p
 # Other designs at the same layer sizes (width, heads, feed-forward), for --design.
 DESIGNS = {"ruvenex": {"1.5b": "ruvenex-1.5b", "7b": "ruvenex-7b"}, "fozerax": {"1.5b": "fozerax-1.5b", "7b": "fozerax-7b"},
            "pefazen": {"1.5b": "pefazen-1.5b", "7b": "pefazen-7b"}, "biravik": {"1.5b": "biravik-1.5b", "7b": "biravik-7b"},
-           "notirax": {"1.5b": "notirax-1.5b", "7b": "notirax-7b"}}
+           "notirax": {"1.5b": "notirax-1.5b", "7b": "notirax-7b"}, "bolelix": {"1.5b": "bolelix-1.5b", "7b": "bolelix-7b"}}
 # the designs a design is measured beside, besides Qwen2: the closest one the engine has
-BESIDE = {"fozerax": ["ruvenex"], "pefazen": ["fozerax"], "biravik": ["fozerax"], "notirax": ["fozerax"]}
+BESIDE = {"fozerax": ["ruvenex"], "pefazen": ["fozerax"], "biravik": ["fozerax"], "notirax": ["fozerax"], "bolelix": ["biravik"]}
 CONFIG = SIZES["1.5b"]
 FALLBACK_PEAKS = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "bf16_tflops_sustained": 1400.0}
 
@@ -475,6 +476,31 @@ def notirax_flops(cfg, T):
     return total + 2 * W * cfg["vocab"]
 
 
+def bolelix_flops(cfg, T):
+    """Arithmetic of a prompt of T tokens through a Bolelix configuration as the design states it: the projections,
+    attention scores and sums over what a query sees, the recurrences' state updates and read-outs, the filters, and the
+    chosen experts only."""
+    W, total = cfg["width"], 0.0
+    for l in cfg["layers"]:
+        m = l["mixer"]
+        H, dv = m["heads"], m["vdim"]
+        if l["type"] == "attention":
+            own = 0 if m.get("kv_from") is not None else m["kv_heads"] * (m["dim"] + dv)
+            total += 2 * T * W * (H * m["dim"] + own + H + H * dv)
+            win = min(T, m["mask"]["size"]) if m.get("mask") else T
+            seen = T * win - win * (win - 1) / 2 + (max(0, T - win) * min(m["mask"].get("keep_first", 0), T) if m.get("mask") else 0)
+            total += 2 * H * (m["dim"] + dv) * seen
+        elif l["type"] == "mamba2":
+            GN = m.get("groups", 1) * m["state"]
+            total += 2 * T * W * (3 * H * dv + 2 * GN + H) + 2 * T * m.get("conv", 1) * (H * dv + 2 * GN) + T * H * m["state"] * dv * 5
+        else:
+            total += 2 * T * W * (2 * H * m["dim"] + 3 * H * dv + 2 * H) + T * H * m["dim"] * (dv + 1) * 5
+        f = l["mlp"]
+        if f:
+            total += 2 * T * W * (3 * f["router"]["top"] * f["expert"]["ff"] + f["router"]["experts"])
+    return total + 2 * W * cfg["vocab"]
+
+
 def design_flops(cfg, T):
     """Arithmetic of a prompt of T tokens through a model of --design's configuration (matrix products, attention
     scores and sums, the recurrence's state updates and read-outs), logits at the last place only."""
@@ -486,6 +512,8 @@ def design_flops(cfg, T):
         return biravik_flops(cfg, T)
     if cfg.get("architecture") == "Notirax":
         return notirax_flops(cfg, T)
+    if cfg.get("architecture") == "Bolelix":
+        return bolelix_flops(cfg, T)
     W, total = cfg["width"], 0.0
     for l in cfg["layers"]:
         a, r = l["mixer"]["left"], l["mixer"]["right"]
