@@ -35,6 +35,7 @@ MODULES: Dict[str, str] = {
     "post": "post_ops.cu",       # norms after the residual sum, per-head query/key norms, mixtures with the token before
     "stream": "stream_ops.cu",   # several residual streams, norms over groups of channels, sinusoidal positions
     "memory": "memory_ops.cu",   # scaled sums with the next norm, state space layers' filters and steps, matrix memories' gates
+    "chunk": "chunk_scan.cu",    # the recurrences of the two lines above over prompt portions, in chunks on the tensor cores
     "talk": "talk_ops.cu",       # attention whose heads exchange their scores before the softmax
     "talk_pf": "talk_prefill.cu",       # the same attention for prompt portions on the tensor cores
     "latent_pf": "latent_prefill.cu",   # the same attention for prompt portions: per-head keys and values, tensor cores

@@ -124,7 +124,7 @@ scaled_sum_norm_kernel(float* __restrict__ x, const float* __restrict__ a, const
 // causal filter over time, y_t = bias + sum_j w[j][c] u_(t - taps + 1 + j) (u before the segment's first row comes from
 // the request's tail, its last taps - 1 inputs, oldest first; zeros for a new request), then silu; and per head, from
 // column dt_col, dt = softplus(raw + dt_bias[h]) and g = exp(-exp(a_log[h]) dt).
-// out rows (ldo): [channels | up to a multiple of 4 | g (H) | dt (H)]. Filter weights tap-major [taps, channels].
+// out rows (ldo): [channels | up to a multiple of 4 | g (H) | dt (H) | ln g (H)]. Filter weights tap-major [taps, channels].
 // inline_tail (steps of one token per request only): the thread that filters a channel, the only reader of its tail, moves it.
 // A CTA of 128 threads: VEC channels a thread, grid (tokens, blocks of channels and heads).
 template <int VEC>
@@ -143,8 +143,10 @@ filter_prepare_kernel(const float* __restrict__ rows, int64_t ld, int col0, int 
         if (h >= n_heads) return;
         const float dt = softplus_(rows[t * ld + dt_col + h] + dt_bias[h]);
         float* o = out + t * ldo + (channels + 3) / 4 * 4;
-        o[h] = expf(-expf(a_log[h]) * dt);
+        const float lng = -expf(a_log[h]) * dt;
+        o[h] = expf(lng);
         o[n_heads + h] = dt;
+        o[2 * n_heads + h] = lng;
         return;
     }
     const int c = u * VEC;
@@ -187,16 +189,16 @@ filter_prepare_kernel(const float* __restrict__ rows, int64_t ld, int col0, int 
 // Gates of a matrix memory over the tokens of every segment in order, one CTA per (segment, head):
 //   i = cap tanh((raw[i_col + h] + i_bias[h]) / cap),   f = log sigmoid(cap tanh((raw[f_col + h] + f_bias[h]) / cap))
 //   m <- max(f + m, i)   (m kept per request and head in `state` [slots, H], zero for a new request)
-//   out rows (ldo): [keep = exp(f + m_before - m) (H) | write = exp(i - m) (H) | floor = exp(-m) (H)]
+//   out rows (ldo): [keep = exp(f + m_before - m) (H) | write = exp(i - m) (H) | floor = exp(-m) (H) | ln keep (H)]
 // The gates and the exponentials are computed in parallel over a tile of tokens; the running maximum walks the tile in
 // one thread, an addition and a maximum a token, so that it does not depend on where a prompt was cut.
 constexpr int GATE_TILE = 512;
 
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(512)
 memory_gates_kernel(const float* __restrict__ rows, int64_t ld, int i_col, int f_col, const float* __restrict__ i_bias,
                     const float* __restrict__ f_bias, float cap, float* __restrict__ state, const int* __restrict__ seg_start,
                     const int* __restrict__ seg_slot, float* __restrict__ out, int64_t ldo, int n_heads, int write_state) {
-    __shared__ __align__(16) float gi[GATE_TILE], gf[GATE_TILE], gm[GATE_TILE + 4];
+    __shared__ __align__(16) float gi[GATE_TILE + 4], gf[GATE_TILE + 4], gm[GATE_TILE + 4];
     ib::pdl_launch_dependents();
     ib::pdl_wait();
     const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
@@ -216,8 +218,11 @@ memory_gates_kernel(const float* __restrict__ rows, int64_t ld, int i_col, int f
         if (tid == 0) {
             // gm[c] is the maximum before token c, gm[n] the one after the tile
             int c = 0;
+            float4 i_next = load4(gi), f_next = load4(gf);   // (four tokens ahead of the walk)
             for (; c + 4 <= n; c += 4) {
-                const float4 i4 = load4(gi + c), f4 = load4(gf + c);
+                const float4 i4 = i_next, f4 = f_next;
+                i_next = load4(gi + c + 4);
+                f_next = load4(gf + c + 4);
                 float4 b4;
                 b4.x = m;
                 m = fmaxf(f4.x + m, i4.x);
@@ -239,9 +244,11 @@ memory_gates_kernel(const float* __restrict__ rows, int64_t ld, int i_col, int f
         for (int c = tid; c < n; c += blockDim.x) {
             float* o = out + (t0 + c0 + c) * ldo;
             const float now = gm[c + 1];
-            o[h] = expf(gf[c] + gm[c] - now);
+            const float lnk = gf[c] + gm[c] - now;
+            o[h] = expf(lnk);
             o[n_heads + h] = expf(gi[c] - now);
             o[2 * n_heads + h] = expf(-now);
+            o[3 * n_heads + h] = lnk;
         }
         m = gm[n];
         __syncthreads();
@@ -281,7 +288,7 @@ IB_EXPORT int ib_filter_prepare(const float* rows, int64_t ld, int col0, int cha
     if (n_tokens <= 0) return IB_OK;
     if (channels <= 0 || taps <= 0 || n_heads <= 0 || !filt_w || !filt_b) return ib::fail(IB_ERR_ARG, "ib_filter_prepare: bad sizes");
     if (taps > 1 && !tails) return ib::fail(IB_ERR_ARG, "ib_filter_prepare: a filter of %d taps needs tails", taps);
-    if (ldo < (channels + 3) / 4 * 4 + 2 * int64_t(n_heads)) return ib::fail(IB_ERR_ARG, "ib_filter_prepare: result rows too short");
+    if (ldo < (channels + 3) / 4 * 4 + 3 * int64_t(n_heads)) return ib::fail(IB_ERR_ARG, "ib_filter_prepare: result rows too short");
     const uintptr_t all = uintptr_t(rows) | uintptr_t(filt_w) | uintptr_t(taps > 1 ? tails : nullptr) | uintptr_t(out);
     const bool vec = channels % 4 == 0 && col0 % 4 == 0 && ld % 4 == 0 && ldo % 4 == 0 && !(all & 15);
     const int units = (vec ? channels / 4 : channels) + n_heads;
@@ -298,11 +305,12 @@ IB_EXPORT int ib_filter_prepare(const float* rows, int64_t ld, int col0, int cha
 
 IB_EXPORT int ib_memory_gates(const float* rows, int64_t ld, int i_col, int f_col, const float* i_bias, const float* f_bias, float cap,
                               float* state, const int* seg_start, const int* seg_slot, float* out, int64_t ldo, int n_segments,
-                              int n_heads, int write_state, cudaStream_t stream) {
+                              int n_heads, int write_state, int max_len, cudaStream_t stream) {
     if (n_segments <= 0) return IB_OK;
-    if (n_heads <= 0 || n_heads > 65535 || !(cap > 0.0f) || ldo < 3 * int64_t(n_heads))
+    if (n_heads <= 0 || n_heads > 65535 || !(cap > 0.0f) || ldo < 4 * int64_t(n_heads))
         return ib::fail(IB_ERR_ARG, "ib_memory_gates: %d heads, a cap of %f", n_heads, double(cap));
-    IB_LAUNCH(memory_gates_kernel, (dim3{unsigned(n_segments), unsigned(n_heads), 1u}), 128, 0, rows, ld, i_col, f_col, i_bias, f_bias, cap,
+    // (the number of threads changes nothing but how many tokens of a tile are formed at a time)
+    IB_LAUNCH(memory_gates_kernel, (dim3{unsigned(n_segments), unsigned(n_heads), 1u}), max_len > 32 ? 512 : 32, 0, rows, ld, i_col, f_col, i_bias, f_bias, cap,
               state, seg_start, seg_slot, out, ldo, n_heads, write_state);
     return ib::check_launch("ib_memory_gates");
 }

@@ -1515,7 +1515,7 @@ def filter_prepare(rows: torch.Tensor, col0: int, filt_w: torch.Tensor, filt_b: 
     """What a state space layer's recurrence reads, from float32 projected rows: columns [col0, col0 + C) each through a
     causal filter (``filt_w`` float32 [taps, C], ``filt_b`` [C], ``tails`` float32 [slots, taps - 1, C]: the inputs before the
     step) and silu; per head, from column dt_col, dt = softplus(raw + dt_bias) and g = exp(-exp(a_log) dt). Returns (float32
-    rows [C | up to a multiple of 4 | g (heads) | dt (heads)], first column of g). ``inline_tail`` (steps of one token per
+    rows [C | up to a multiple of 4 | g (heads) | dt (heads) | ln g (heads)], first column of g). ``inline_tail`` (steps of one token per
     request only): the kernel also moves the tails (no ``tail_update``)."""
     _check(rows, "rows", torch.float32)
     T, ld = rows.shape
@@ -1532,7 +1532,7 @@ def filter_prepare(rows: torch.Tensor, col0: int, filt_w: torch.Tensor, filt_b: 
         if tuple(tails.shape[1:]) != (taps - 1, C):
             raise KernelError(f"tails must be [slots, {taps - 1}, {C}], got {tuple(tails.shape)}")
     g_col = -(-C // 4) * 4
-    out = torch.empty((T, -(-(g_col + 2 * H) // 4) * 4), dtype=torch.float32, device=rows.device)
+    out = torch.empty((T, -(-(g_col + 3 * H) // 4) * 4), dtype=torch.float32, device=rows.device)
     f = _fn("memory", "ib_filter_prepare", [c_void_p, c_int64, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p,
                                             c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int64, c_void_p])
     _call(f, rows.data_ptr(), ld, int(col0), C, filt_w.data_ptr(), filt_b.data_ptr(), taps, _ptr(tails) if taps > 1 else None,
@@ -1545,7 +1545,8 @@ def memory_gates(rows: torch.Tensor, i_col: int, f_col: int, i_bias: torch.Tenso
                  step, write_state: bool = True) -> torch.Tensor:
     """Gates of a matrix memory over the tokens of every segment in order, from float32 projected rows: with
     i = cap tanh((raw_i + i_bias) / cap) and f = log sigmoid(cap tanh((raw_f + f_bias) / cap)) per head, m <- max(f + m, i)
-    (kept in ``state`` float32 [slots, heads]). Returns float32 [T, exp(f + m_before - m) | exp(i - m) | exp(-m)], heads each."""
+    (kept in ``state`` float32 [slots, heads]). Returns float32 [T, exp(f + m_before - m) | exp(i - m) | exp(-m) | f + m_before - m],
+    heads each."""
     _check(rows, "rows", torch.float32)
     T, ld = rows.shape
     H = i_bias.numel()
@@ -1554,9 +1555,53 @@ def memory_gates(rows: torch.Tensor, i_col: int, f_col: int, i_bias: torch.Tenso
     _check(state, "state", torch.float32, (state.shape[0], H))
     if min(i_col, f_col) < 0 or max(i_col, f_col) + H > ld:
         raise KernelError("memory_gates: columns lie outside the rows")
-    out = torch.empty((T, 3 * H), dtype=torch.float32, device=rows.device)
+    out = torch.empty((T, 4 * H), dtype=torch.float32, device=rows.device)
     f = _fn("memory", "ib_memory_gates", [c_void_p, c_int64, c_int, c_int, c_void_p, c_void_p, c_float] + [c_void_p] * 4 +
-            [c_int64, c_int, c_int, c_int, c_void_p])
+            [c_int64, c_int, c_int, c_int, c_int, c_void_p])
     _call(f, rows.data_ptr(), ld, int(i_col), int(f_col), i_bias.data_ptr(), f_bias.data_ptr(), float(cap), state.data_ptr(),
-          step.seg_start.data_ptr(), step.seg_slot.data_ptr(), out.data_ptr(), 3 * H, step.seg_slot.numel(), H, int(write_state), _stream())
+          step.seg_start.data_ptr(), step.seg_slot.data_ptr(), out.data_ptr(), 4 * H, step.seg_slot.numel(), H, int(write_state), int(step.max_q_len), _stream())
     return out
+
+
+CHUNK_SCAN_FROM = 24          # segments of more tokens than this are worth the chunked form
+
+
+def step_scan(rows: torch.Tensor, q_col: int, k_col: int, v_col: int, aux: torch.Tensor, g_col: int, b_col: int, lng_col: int,
+              state: torch.Tensor, step, n_heads: int, heads_per_qk: int, dim: int, v_dim: int, write_state: bool = True,
+              skip: Optional[torch.Tensor] = None, ones_state: Optional[torch.Tensor] = None, chunked: bool = False):
+    """S <- g S + b k v^T, o = S^T q + skip v per head over the tokens of every segment in order, with g, b and ln g per head
+    and token in columns of the float32 rows ``aux`` (g and b side by side for the token-by-token form). ``chunked`` (where q,
+    k and v may be rounded to bfloat16): steps with long segments go through the form that takes 64 tokens at a time on
+    the tensor cores, where the sizes allow; all else token by token (``state_scan`` SCAN_STEP, see there). Returns o float32
+    [T, heads * v_dim], with ``ones_state`` (o, n.q)."""
+    if not (chunked and step.max_q_len >= CHUNK_SCAN_FROM and dim <= int(_fn("chunk", "ib_chunk_scan_max_dim", [])())):
+        if b_col != g_col + n_heads:
+            raise KernelError("the token-by-token form reads decays and strengths side by side")
+        return state_scan(SCAN_STEP, rows, q_col, k_col, v_col, aux, g_col, state, step.seg_start, step.seg_slot, n_heads, heads_per_qk, dim,
+                          v_dim, write_state, step.max_q_len, bonus=skip, ones_state=ones_state)
+    _check(rows, "rows", torch.float32)
+    _check(aux, "aux", torch.float32)
+    _check(state, "state", torch.float32)
+    T, ld = rows.shape
+    n_qk = n_heads // heads_per_qk
+    if tuple(state.shape[1:]) != (n_heads, dim, v_dim):
+        raise KernelError(f"state must be [slots, {n_heads}, {dim}, {v_dim}], got {tuple(state.shape)}")
+    if min(q_col, k_col, v_col) < 0 or max(q_col, k_col) + n_qk * dim > ld or v_col + n_heads * v_dim > ld:
+        raise KernelError("the q, k or v columns lie outside the rows")
+    if aux.shape[0] != T or min(b_col, lng_col) < 0 or max(b_col, lng_col) + n_heads > aux.shape[1]:
+        raise KernelError("the decay columns lie outside their rows")
+    if skip is not None:
+        _check(skip, "skip", torch.float32, (n_heads,))
+    ones_out = None
+    if ones_state is not None:
+        _check(ones_state, "ones_state", torch.float32, (state.shape[0], n_heads, dim))
+        ones_out = torch.empty((T, n_heads), dtype=torch.float32, device=rows.device)
+    S = step.seg_slot.numel()
+    _check(step.seg_start, "seg_start", torch.int32, (S + 1,))
+    out = torch.empty((T, n_heads * v_dim), dtype=torch.float32, device=rows.device)
+    f = _fn("chunk", "ib_chunk_scan", [c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_int64, c_int, c_int] + [c_void_p] * 7 +
+            [c_int] * 7 + [c_void_p])
+    _call(f, rows.data_ptr(), ld, int(q_col), int(k_col), int(v_col), aux.data_ptr(), aux.shape[1], int(b_col), int(lng_col), state.data_ptr(),
+          _ptr(ones_state), step.seg_start.data_ptr(), step.seg_slot.data_ptr(), out.data_ptr(), _ptr(ones_out), _ptr(skip), S, n_heads,
+          int(heads_per_qk), dim, v_dim, int(write_state), torch.cuda.get_device_properties(rows.device).multi_processor_count, _stream())
+    return out if ones_state is None else (out, ones_out)

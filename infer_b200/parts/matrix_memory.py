@@ -98,8 +98,8 @@ class MatrixMemory(Mixer):
         rows, c0 = own_or_projected(self, x, self.proj, torch.float32)
         gate_col = c0 + 2 * nq + nv
         gates = ops.memory_gates(rows, gate_col + nv, gate_col + nv + H, self.input_b, self.forget_b, self.cap, cache["m"], step, write_cache)
-        o, den = ops.state_scan(ops.SCAN_STEP, rows, c0, c0 + nq, c0 + 2 * nq, gates, 0, cache["S"], step.seg_start, step.seg_slot, H, 1,
-                                self.dim, self.v_dim, write_cache, step.max_q_len, ones_state=cache["n"])
+        o, den = ops.step_scan(rows, c0, c0 + nq, c0 + 2 * nq, gates, 0, H, 3 * H, cache["S"], step, H, 1, self.dim, self.v_dim, write_cache,
+                               ones_state=cache["n"], chunked=self.rt.dtype == torch.bfloat16)
         # (the read-outs are linear in q: its constant is applied to them)
         y = ops.group_norm_gate(o, self.norm_w, self.eps, rows, gate_col, "sigmoid", H, self.v_dim, self.rt.dtype, den=den,
                                 den_floor=gates, floor_col=2 * H, den_mult=float(self.dim) ** -0.5, den_eps=self.floor)

@@ -118,8 +118,9 @@ class StateSpace(Mixer):
             ops.tail_update(rows, u_col, tails, step.seg_start, step.seg_slot)
         k_col = self.inner
         q_col = k_col + self.groups * self.state
-        o = ops.state_scan(ops.SCAN_STEP, prep, q_col, k_col, 0, prep, g_col, cache["S"], step.seg_start, step.seg_slot, self.n_heads,
-                           self.n_heads // self.groups, self.state, self.v_dim, write_cache, step.max_q_len, bonus=self.skip)
+        o = ops.step_scan(prep, q_col, k_col, 0, prep, g_col, g_col + self.n_heads, g_col + 2 * self.n_heads, cache["S"], step, self.n_heads,
+                          self.n_heads // self.groups, self.state, self.v_dim, write_cache, skip=self.skip,
+                          chunked=self.rt.dtype == torch.bfloat16)
         y = ops.group_norm_gate(o, self.norm_w, self.eps, rows, c0, "silu", self.norm_groups, self.inner // self.norm_groups,
                                 self.rt.dtype, gate_first=True)
         if residual is None:

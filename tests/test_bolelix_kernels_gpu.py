@@ -257,6 +257,46 @@ def test_step_scan_cuttings_are_bit_equal():
         assert torch.equal(o, outs[0])
 
 
+@pytest.mark.parametrize("sizes", [(2, 2, 16, 32), (4, 2, 40, 20), (3, 1, 5, 9), (2, 1, 128, 64), (24, 2, 128, 128), (5, 1, 33, 3), (6, 3, 64, 24), (12, 12, 64, 128)])
+@pytest.mark.parametrize("ones", [False, True], ids=["values", "ones"])
+def test_scan_in_chunks_on_the_tensor_cores_over_steps(sizes, ones):
+    """Segments around multiples of 64 tokens beside short ones, the state carried from chunked steps to single tokens and
+    back; decays of 0 and 1e-30 among them. Inputs are bfloat16 numbers: the chunked form then rounds nothing of them, and
+    agrees with the exact recurrence to the sixteen bits that it keeps of states and scores."""
+    H, G, d, dv = sizes
+    total = (330, 276)
+    seqs = _step_case(H, G, d, dv, d + dv, total)
+    for x in seqs.values():
+        for n in "qkv":
+            x[n] = x[n].to(torch.bfloat16).float()
+        x["g"][:] = torch.where(x["g"] > 1e-20, x["g"] ** 0.1, x["g"])            # (states that hold many tokens)
+    skip = torch.linspace(-1, 1, H)
+    ref = _step_reference(seqs, H, G, skip)
+    state = torch.full((3, H, d, dv), float("nan"), device=DEV)
+    n_state = torch.full((3, H, d), float("nan"), device=DEV)
+    for t in (state, n_state):
+        t[0].zero_(), t[2].zero_()
+    at = {0: 0, 2: 0}
+    before = ops.LAUNCH_KINDS["ib_chunk_scan"]
+    steps = ([100, 63], [1, 1], [64, 128], [2, 65], [128, 1], [33, 16], [2, 2])
+    for lens in steps:
+        step = _Step(lens, [at[0], at[2]], [0, 2])
+        step.max_q_len = max(lens)
+        rows, aux = _step_rows(seqs, at, lens)
+        got = ops.step_scan(rows, 4, 4 + G * d, 4 + 2 * G * d, aux, 1, 1 + H, 1 + 2 * H, state, step, H, H // G, d, dv, True,
+                            skip=skip.to(DEV), ones_state=n_state if ones else None, chunked=True)
+        o, n = got if ones else (got, None)
+        want = [torch.cat([ref[s][i][at[s]:at[s] + m] for s, m in zip((0, 2), lens)]) for i in range(2)]
+        size = float(want[0].abs().max())
+        assert torch.allclose(o.double().cpu().view(-1, H, dv), want[0], rtol=2e-4, atol=4e-5 * size), lens
+        if ones:
+            assert torch.allclose(n.double().cpu(), want[1], rtol=2e-4, atol=4e-5 * float(want[1].abs().max()))
+        for s, m in zip((0, 2), lens):
+            at[s] += m
+    assert ops.LAUNCH_KINDS["ib_chunk_scan"] - before == sum(max(l) >= ops.CHUNK_SCAN_FROM for l in steps)
+    assert (at[0], at[2]) == total and bool(torch.isnan(state[1]).all()) and bool(torch.isnan(n_state[1]).all())
+
+
 @pytest.mark.parametrize("size,groups", [(7, 3), (24, 1), (64, 2), (768, 2), (2000, 1)])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16], ids=["f32", "bf16"])
 def test_gate_in_front_of_a_norm_over_groups(size, groups, dtype):
@@ -294,7 +334,10 @@ def test_memory_gates_over_steps(H, cap):
         for lens in all_lens:
             step = _Step(lens, [at[0], at[2]], [0, 2])
             rows = d(torch.cat([seqs[s][at[s]:at[s] + m] for s, m in zip((0, 2), lens)]))
-            got = ops.memory_gates(rows, 2, 2 + H, d(bi), d(bf), cap, state, step).cpu()[:, :3 * H]
+            step.max_q_len = max(lens)
+            got = ops.memory_gates(rows, 2, 2 + H, d(bi), d(bf), cap, state, step).cpu()
+            assert torch.allclose(got[:, 3 * H:].exp(), got[:, :H], rtol=1e-6)
+            got = got[:, :3 * H]
             outs[0].append(got[:lens[0]]), outs[2].append(got[lens[0]:])
             for s, m in zip((0, 2), lens):
                 at[s] += m
