@@ -185,6 +185,77 @@ filter_prepare_kernel(const float* __restrict__ rows, int64_t ld, int col0, int 
     }
 }
 
+// filter_prepare for FT tokens a thread (prompt portions): the inputs that neighbouring tokens share are read once. Tokens
+// near their segment's start, or of different segments, take their inputs one by one as above; the sums are the same.
+constexpr int FT = 4;
+
+template <int TAPS>
+__global__ void __launch_bounds__(128)
+filter_prepare_tokens_kernel(const float* __restrict__ rows, int64_t ld, int col0, int channels, const float* __restrict__ filt_w,
+                             const float* __restrict__ filt_b, const float* __restrict__ tails, int dt_col, const float* __restrict__ dt_bias,
+                             const float* __restrict__ a_log, int n_heads, const int* __restrict__ token_seg,
+                             const int* __restrict__ seg_start, const int* __restrict__ seg_slot, float* __restrict__ out, int64_t ldo,
+                             int64_t n_tokens) {
+    ib::pdl_launch_dependents();
+    ib::pdl_wait();
+    const int64_t t0 = int64_t(blockIdx.x) * FT;
+    const int nt = int(min(int64_t(FT), n_tokens - t0));
+    const int u = blockIdx.y * blockDim.x + threadIdx.x;
+    const int n_units = channels / 4;
+    if (u >= n_units) {
+        const int h = u - n_units;
+        if (h >= n_heads) return;
+        const float rate = expf(a_log[h]);
+        for (int i = 0; i < nt; i++) {
+            const float dt = softplus_(rows[(t0 + i) * ld + dt_col + h] + dt_bias[h]);
+            float* o = out + (t0 + i) * ldo + channels;
+            const float lng = -rate * dt;
+            o[h] = expf(lng);
+            o[n_heads + h] = dt;
+            o[2 * n_heads + h] = lng;
+        }
+        return;
+    }
+    const int c = u * 4;
+    float4 w[TAPS];
+#pragma unroll
+    for (int j = 0; j < TAPS; j++) w[j] = load4(filt_w + int64_t(j) * channels + c);
+    const float4 b = load4(filt_b + c);
+    auto finish = [&](int64_t t, float4 y) { store4(out + t * ldo + c, make_float4(silu_(y.x), silu_(y.y), silu_(y.z), silu_(y.w))); };
+    const int s = token_seg[t0];
+    const int first = int(t0 - seg_start[s]);
+    if (nt == FT && first >= TAPS - 1 && token_seg[t0 + FT - 1] == s) {
+        float4 in[FT + TAPS - 1];
+#pragma unroll
+        for (int i = 0; i < FT + TAPS - 1; i++) in[i] = load4(rows + (t0 - (TAPS - 1) + i) * ld + col0 + c);
+#pragma unroll
+        for (int i = 0; i < FT; i++) {
+            float4 y = b;
+#pragma unroll
+            for (int j = 0; j < TAPS; j++) {
+                y.x = fmaf(w[j].x, in[i + j].x, y.x); y.y = fmaf(w[j].y, in[i + j].y, y.y);
+                y.z = fmaf(w[j].z, in[i + j].z, y.z); y.w = fmaf(w[j].w, in[i + j].w, y.w);
+            }
+            finish(t0 + i, y);
+        }
+        return;
+    }
+    for (int i = 0; i < nt; i++) {
+        const int64_t t = t0 + i;
+        const int sg = token_seg[t];
+        const int i_local = int(t - seg_start[sg]);
+        const float* tail = TAPS > 1 ? tails + int64_t(seg_slot[sg]) * (TAPS - 1) * channels + c : nullptr;
+        float4 y = b;
+#pragma unroll
+        for (int j = 0; j < TAPS; j++) {
+            const int back = TAPS - 1 - j;
+            const float4 v = load4(i_local >= back ? rows + (t - back) * ld + col0 + c : tail + int64_t(TAPS - 1 + i_local - back) * channels);
+            y.x = fmaf(w[j].x, v.x, y.x); y.y = fmaf(w[j].y, v.y, y.y); y.z = fmaf(w[j].z, v.z, y.z); y.w = fmaf(w[j].w, v.w, y.w);
+        }
+        finish(t, y);
+    }
+}
+
 // ------------------------------------------------------------------------------------------------
 // Gates of a matrix memory over the tokens of every segment in order, one CTA per (segment, head):
 //   i = cap tanh((raw[i_col + h] + i_bias[h]) / cap),   f = log sigmoid(cap tanh((raw[f_col + h] + f_bias[h]) / cap))
@@ -294,6 +365,15 @@ IB_EXPORT int ib_filter_prepare(const float* rows, int64_t ld, int col0, int cha
     const int units = (vec ? channels / 4 : channels) + n_heads;
     const dim3 grid{unsigned(n_tokens), blocks_for(units, 128), 1u};
     if (grid.y > 65535) return ib::fail(IB_ERR_ARG, "ib_filter_prepare: too many channels");
+    if (vec && !inline_tail && taps <= 4 && n_tokens >= 256) {          // (the same sums for a token, fewer reads)
+        const dim3 grid4{blocks_for(n_tokens, FT), grid.y, 1u};
+#define IB_FT(TT)                                                                                                                     \
+        IB_LAUNCH(filter_prepare_tokens_kernel<TT>, grid4, 128, 0, rows, ld, col0, channels, filt_w, filt_b, tails, dt_col, dt_bias, a_log, \
+                  n_heads, token_seg, seg_start, seg_slot, out, ldo, n_tokens)
+        if (taps == 1) IB_FT(1); else if (taps == 2) IB_FT(2); else if (taps == 3) IB_FT(3); else IB_FT(4);
+#undef IB_FT
+        return ib::check_launch("ib_filter_prepare");
+    }
     if (vec)
         IB_LAUNCH(filter_prepare_kernel<4>, grid, 128, 0, rows, ld, col0, channels, filt_w, filt_b, taps, tails, inline_tail, dt_col, dt_bias,
                   a_log, n_heads, token_seg, seg_start, seg_slot, out, ldo);

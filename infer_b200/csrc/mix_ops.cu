@@ -182,24 +182,36 @@ __global__ void glu_act_vec_kernel(const bf16* __restrict__ rows, int64_t ld, in
     *reinterpret_cast<uint4*>(out + i * 8) = res;
 }
 
+template <typename T>
+__device__ __forceinline__ void load8(const T* p, float (&x)[8]);
+template <>
+__device__ __forceinline__ void load8<float>(const float* p, float (&x)[8]) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
+}
+template <>
+__device__ __forceinline__ void load8<bf16>(const bf16* p, float (&x)[8]) {
+    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const float2 f = __bfloat1622float2(h[i]);
+        x[2 * i] = f.x;
+        x[2 * i + 1] = f.y;
+    }
+}
+
 // ------------------------------------------------------------------------------------------------
 // Router: scores = softmax(logits) over all experts, or the logits' sigmoids; experts form n_groups groups of neighbours,
 // a group's score is its largest, or the sum of its two largest (of its one, if it has one); only experts of the `keep`
 // best groups can be chosen; the `top` largest of those are chosen (ties: the lower index); their weights are their
 // scores divided by (their sum + sum_eps), or as they are, times `mult`. One warp per token.
 // weights [tokens, experts]: a chosen expert's weight, zero elsewhere. chosen [tokens, top] (optional): the indices.
-__global__ void __launch_bounds__(128)
-route_kernel(const float* __restrict__ logits, int64_t n_tokens, int n_experts, int top, int n_groups, int keep,
-             float sum_eps, int sigmoid, int group_best, int renormalise, float mult, float* __restrict__ weights,
-             int* __restrict__ chosen) {
-    ib::pdl_wait();
-    extern __shared__ float sm[];
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int64_t t = int64_t(blockIdx.x) * (blockDim.x >> 5) + warp;
-    if (t >= n_tokens) return;
-    float* s = sm + warp * (n_experts + n_groups);          // scores; a chosen expert's score becomes -(1 + score)
-    float* gs = s + n_experts;                               // group scores; -1: a kept group, -2: not kept
-    const float* z = logits + t * n_experts;
+// s [experts]: scores; a chosen expert's score becomes -(1 + score). gs [groups]: group scores; -1: a kept group, -2: not
+// kept. Both in shared memory, the warp's own; z: the token's logits (may be s itself).
+__device__ __forceinline__ void route_token(const float* z, float* s, float* gs, int64_t t, int lane, int n_experts, int top, int n_groups,
+                                            int keep, float sum_eps, int sigmoid, int group_best, int renormalise, float mult,
+                                            float* __restrict__ weights, int* __restrict__ chosen) {
     if (sigmoid) {
         for (int e = lane; e < n_experts; e += 32) s[e] = sigmoid_(z[e]);
     } else {
@@ -268,6 +280,60 @@ route_kernel(const float* __restrict__ logits, int64_t n_tokens, int n_experts, 
     for (int e = lane; e < n_experts; e += 32) weights[t * n_experts + e] = s[e] < 0.0f ? (-1.0f - s[e]) * inv : 0.0f;
 }
 
+__global__ void __launch_bounds__(128)
+route_kernel(const float* __restrict__ logits, int64_t n_tokens, int n_experts, int top, int n_groups, int keep,
+             float sum_eps, int sigmoid, int group_best, int renormalise, float mult, float* __restrict__ weights,
+             int* __restrict__ chosen) {
+    ib::pdl_wait();
+    extern __shared__ float sm[];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int64_t t = int64_t(blockIdx.x) * (blockDim.x >> 5) + warp;
+    if (t >= n_tokens) return;
+    float* s = sm + warp * (n_experts + n_groups);
+    route_token(logits + t * n_experts, s, s + n_experts, t, lane, n_experts, top, n_groups, keep, sum_eps, sigmoid, group_best, renormalise,
+                mult, weights, chosen);
+}
+
+// The same with the router's product in front of it: logits = W x in float, rows and matrix in storage T (widths of whole
+// 16-byte pieces, up to EB experts). One warp per token, its lanes along the row; a token's sums do not depend on the others.
+template <typename T, int EB>
+__global__ void __launch_bounds__(128)
+route_rows_kernel(const T* __restrict__ x, const T* __restrict__ w, int64_t n_tokens, int width, int n_experts, int top, int n_groups,
+                  int keep, float sum_eps, int sigmoid, int group_best, int renormalise, float mult, float* __restrict__ weights,
+                  int* __restrict__ chosen) {
+    ib::pdl_wait();
+    extern __shared__ float sm[];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int64_t t = int64_t(blockIdx.x) * (blockDim.x >> 5) + warp;
+    if (t >= n_tokens) return;
+    float* s = sm + warp * (n_experts + n_groups);
+    float acc[EB];
+#pragma unroll
+    for (int e = 0; e < EB; e++) acc[e] = 0.0f;
+    for (int i = lane * 8; i < width; i += 256) {
+        float xv[8];
+        load8<T>(x + t * width + i, xv);
+#pragma unroll
+        for (int e = 0; e < EB; e++) {
+            if (e < n_experts) {
+                float wv[8];
+                load8<T>(w + int64_t(e) * width + i, wv);
+#pragma unroll
+                for (int j = 0; j < 8; j++) acc[e] = fmaf(xv[j], wv[j], acc[e]);
+            }
+        }
+    }
+#pragma unroll
+    for (int e = 0; e < EB; e++) {
+        if (e < n_experts) {
+            const float z = ib::warp_sum(acc[e]);
+            if (lane == e % 32) s[e] = z;
+        }
+    }
+    __syncwarp();
+    route_token(s, s, s + n_experts, t, lane, n_experts, top, n_groups, keep, sum_eps, sigmoid, group_best, renormalise, mult, weights, chosen);
+}
+
 // ------------------------------------------------------------------------------------------------
 // In front of paged attention: projected rows [q | k | v] (q at column col0) -> q rows for the attention kernel, k and
 // v into the token's page. q is normalised over ALL its heads * d channels at once, with a weight per channel (wq),
@@ -327,25 +393,6 @@ rownorm_store_kernel(const T* __restrict__ rows, int64_t ld, int col0, const flo
 constexpr int KC = 128;
 constexpr int GMAX = 16;
 constexpr int VT = 32;                 // value rows staged at a time
-
-template <typename T>
-__device__ __forceinline__ void load8(const T* p, float (&x)[8]);
-template <>
-__device__ __forceinline__ void load8<float>(const float* p, float (&x)[8]) {
-    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-    x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
-}
-template <>
-__device__ __forceinline__ void load8<bf16>(const bf16* p, float (&x)[8]) {
-    const uint4 u = *reinterpret_cast<const uint4*>(p);
-    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
-#pragma unroll
-    for (int i = 0; i < 4; i++) {
-        const float2 f = __bfloat1622float2(h[i]);
-        x[2 * i] = f.x;
-        x[2 * i + 1] = f.y;
-    }
-}
 
 // GB: the group's size rounded up to 1, 2, 4, 8 or 16 (the loops over a group's heads are unrolled to it).
 template <typename T, int GB>
@@ -1199,6 +1246,35 @@ IB_EXPORT int ib_route(const float* logits, int64_t n_tokens, int n_experts, int
     IB_LAUNCH(route_kernel, blocks_for(n_tokens, 4), 128, smem, logits, n_tokens, n_experts, top, n_groups, keep, sum_eps,
               sigmoid, group_best, renormalise, mult, weights, chosen);
     return ib::check_launch("ib_route");
+}
+
+// The most experts that ib_route_rows takes.
+IB_EXPORT int ib_route_rows_max_experts() { return 64; }
+
+// ib_route with the router's product in front: x [tokens, width], w [experts, width] in one storage dtype.
+IB_EXPORT int ib_route_rows(const void* x, const void* w, int64_t n_tokens, int width, int n_experts, int top, int n_groups, int keep,
+                            float sum_eps, int sigmoid, int group_best, int renormalise, float mult, float* weights, int* chosen, int dtype,
+                            cudaStream_t stream) {
+    if (n_tokens <= 0) return IB_OK;
+    if (n_experts <= 0 || n_experts > 64 || n_groups <= 0 || n_experts % n_groups || keep <= 0 || keep > n_groups || top <= 0 ||
+        top > keep * (n_experts / n_groups) || (group_best != 1 && group_best != 2))
+        return ib::fail(IB_ERR_ARG, "ib_route_rows: %d experts in %d groups, %d kept, %d chosen", n_experts, n_groups, keep, top);
+    if (width <= 0 || width % 8 || ((uintptr_t(x) | uintptr_t(w)) & 15)) return ib::fail(IB_ERR_ARG, "ib_route_rows: rows of %d are not whole 16-byte pieces", width);
+    const size_t smem = size_t(4) * (n_experts + n_groups) * sizeof(float);
+    const int eb = n_experts <= 8 ? 8 : (n_experts <= 16 ? 16 : (n_experts <= 32 ? 32 : 64));
+#define IB_RR(TT, EE)                                                                                                                \
+    IB_LAUNCH((route_rows_kernel<TT, EE>), blocks_for(n_tokens, 4), 128, smem, (const TT*)x, (const TT*)w, n_tokens, width, n_experts, \
+              top, n_groups, keep, sum_eps, sigmoid, group_best, renormalise, mult, weights, chosen)
+#define IB_RR_BY(TT)                                                                                                                 \
+    do {                                                                                                                             \
+        if (eb == 8) IB_RR(TT, 8); else if (eb == 16) IB_RR(TT, 16); else if (eb == 32) IB_RR(TT, 32); else IB_RR(TT, 64);           \
+    } while (0)
+    if (dtype == IB_F32) IB_RR_BY(float);
+    else if (dtype == IB_BF16) IB_RR_BY(bf16);
+    else return ib::fail(IB_ERR_ARG, "ib_route_rows: unknown dtype %d", dtype);
+#undef IB_RR_BY
+#undef IB_RR
+    return ib::check_launch("ib_route_rows");
 }
 
 IB_EXPORT int ib_rownorm_store(const void* rows, int64_t ld, int col0, const float* wq, const float* wk, float eps,

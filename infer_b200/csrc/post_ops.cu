@@ -155,6 +155,24 @@ __global__ void gate_mul_kernel(T* __restrict__ ctx, const T* __restrict__ rows,
     ctx[i] = ib::from_f32<T>(ib::to_f32(ctx[i]) * sigmoid_(ib::to_f32(rows[t * ld + gate_col + (per > 1 ? c / per : c)])));
 }
 
+// The same for bfloat16 rows whose sizes and addresses allow 16-byte accesses: eight channels a thread (they share a gate).
+__global__ void gate_mul_vec_kernel(bf16* __restrict__ ctx, const bf16* __restrict__ rows, int64_t ld, int64_t gate_col, int64_t width8,
+                                    int64_t per8, int64_t n8) {
+    ib::pdl_wait();
+    const int64_t i = int64_t(blockIdx.x) * blockDim.x + threadIdx.x;
+    if (i >= n8) return;
+    const int64_t t = i / width8, c = i - t * width8;
+    const float g = sigmoid_(ib::to_f32(rows[t * ld + gate_col + c / per8]));
+    uint4 u = *reinterpret_cast<const uint4*>(ctx + i * 8);
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&u);
+#pragma unroll
+    for (int k = 0; k < 4; k++) {
+        const float2 f = __bfloat1622float2(h[k]);
+        h[k] = __floats2bfloat162_rn(f.x * g, f.y * g);
+    }
+    *reinterpret_cast<uint4*>(ctx + i * 8) = u;
+}
+
 // silu of columns [col0, col0 + width) of float rows, in place.
 __global__ void silu_rows_kernel(float* __restrict__ rows, int64_t ld, int64_t col0, int64_t width, int64_t n) {
     ib::pdl_wait();
@@ -324,6 +342,67 @@ group_norm_gate_wide_kernel(const float* __restrict__ o, const float* __restrict
     }
 }
 
+// group_norm_gate where sizes and addresses allow four channels an access: one warp per (token, group) of up to 128 * PIECES
+// channels, which it keeps in registers between the sum of squares and the result.
+__device__ __forceinline__ float4 load4_(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4_(const bf16* p) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void store4_(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4_(bf16* p, float4 v) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const unsigned*>(&lo), *reinterpret_cast<const unsigned*>(&hi));
+}
+__device__ __forceinline__ float acted(float z, int act) { return act == 1 ? silu_(z) : (act == 2 ? sigmoid_(z) : z); }
+
+template <typename TG, typename TOut, int PIECES>
+__global__ void __launch_bounds__(256)
+group_norm_gate_vec_kernel(const float* __restrict__ o, const float* __restrict__ w, float eps, const TG* __restrict__ gate, int64_t ldg,
+                           int64_t gate_col, int act, TOut* __restrict__ out, int64_t n_rows, int n_groups, int size, int gate_first,
+                           const GroupScale scale) {
+    ib::pdl_wait();
+    const int lane = threadIdx.x & 31;
+    const int64_t r = int64_t(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (r >= n_rows) return;
+    const int64_t t = r / n_groups;
+    const int g = int(r - t * n_groups);
+    const float* x = o + r * size;
+    const TG* z = gate ? gate + t * ldg + gate_col + int64_t(g) * size : nullptr;
+    float4 v[PIECES], m[PIECES];
+#pragma unroll
+    for (int i = 0; i < PIECES; i++) {
+        const int j = (i * 32 + lane) * 4;
+        v[i] = j < size ? load4_(x + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+        m[i] = z && j < size ? load4_(z + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    const float pre = scale.at(t, g, n_groups);
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < PIECES; i++) {
+        if (z) { m[i].x = acted(m[i].x, act); m[i].y = acted(m[i].y, act); m[i].z = acted(m[i].z, act); m[i].w = acted(m[i].w, act); }
+        v[i].x *= pre; v[i].y *= pre; v[i].z *= pre; v[i].w *= pre;
+        float4 p = v[i];
+        if (gate_first) { p.x *= m[i].x; p.y *= m[i].y; p.z *= m[i].z; p.w *= m[i].w; }
+        ss = fmaf(p.x, p.x, ss); ss = fmaf(p.y, p.y, ss); ss = fmaf(p.z, p.z, ss); ss = fmaf(p.w, p.w, ss);
+    }
+    ss = ib::warp_sum(ss);
+    const float f = 1.0f / sqrtf(ss / float(size) + eps);
+#pragma unroll
+    for (int i = 0; i < PIECES; i++) {
+        const int j = (i * 32 + lane) * 4;
+        if (j >= size) continue;
+        float4 y = make_float4(v[i].x * f, v[i].y * f, v[i].z * f, v[i].w * f);
+        if (w) {
+            const float4 ww = load4_(w + int64_t(g) * size + j);
+            y.x *= ww.x; y.y *= ww.y; y.z *= ww.z; y.w *= ww.w;
+        }
+        if (z) { y.x *= m[i].x; y.y *= m[i].y; y.z *= m[i].z; y.w *= m[i].w; }
+        store4_(out + r * size + j, y);
+    }
+}
+
 // double_exp_decay for TT tokens a CTA: a thread keeps one channel's column of `up` in flight once for all of them.
 constexpr int DECAY_TOKENS = 8;
 template <typename T>
@@ -403,6 +482,8 @@ IB_EXPORT int ib_gate_mul(void* ctx, const void* rows, int64_t ld, int64_t gate_
     const int64_t n = n_tokens * width;
     if (n <= 0) return IB_OK;
     if (dtype == IB_F32) IB_LAUNCH(gate_mul_kernel<float>, blocks_for(n, 256), 256, 0, (float*)ctx, (const float*)rows, ld, gate_col, width, per, n);
+    else if (dtype == IB_BF16 && per > 1 && per % 8 == 0 && width % per == 0 && !(uintptr_t(ctx) & 15))
+        IB_LAUNCH(gate_mul_vec_kernel, blocks_for(n / 8, 256), 256, 0, (bf16*)ctx, (const bf16*)rows, ld, gate_col, width / 8, per / 8, n / 8);
     else if (dtype == IB_BF16) IB_LAUNCH(gate_mul_kernel<bf16>, blocks_for(n, 256), 256, 0, (bf16*)ctx, (const bf16*)rows, ld, gate_col, width, per, n);
     else return ib::fail(IB_ERR_ARG, "ib_gate_mul: unknown dtype %d", dtype);
     return ib::check_launch("ib_gate_mul");
@@ -469,11 +550,19 @@ IB_EXPORT int ib_group_norm_gate(const float* o, const float* w, float eps, cons
     if (gate_first && !gate) return ib::fail(IB_ERR_ARG, "ib_group_norm_gate: a gate in front of the norm needs its logits");
     if (den && !den_floor) return ib::fail(IB_ERR_ARG, "ib_group_norm_gate: a denominator needs its lower bound");
     const GroupScale scale{den, den_floor, ldf, floor_col, den_mult, den_eps};
-    const bool wide = size >= 512;                          // (by the group's size only, never by the number of rows)
+    // (the form goes by sizes and addresses only, never by the number of rows)
+    const bool vec = size % 4 == 0 && size <= 1024 && !((uintptr_t(o) | uintptr_t(w) | uintptr_t(out)) & 15) &&
+                     (!gate || (!(uintptr_t(gate) & 15) && ldg % 4 == 0 && gate_col % 4 == 0));
+    const bool wide = !vec && size >= 512;
     const unsigned grid = wide ? unsigned(rows) : blocks_for(rows, 8);
+#define IB_GNV(TG, TO, PP) IB_LAUNCH((group_norm_gate_vec_kernel<TG, TO, PP>), grid, 256, 0, o, w, eps, (const TG*)gate, ldg, gate_col, act, (TO*)out, rows, n_groups, size, gate_first, scale)
 #define IB_GN(TG, TO)                                                                                                               \
     do {                                                                                                                            \
-        if (wide) IB_LAUNCH((group_norm_gate_wide_kernel<TG, TO>), grid, 256, 0, o, w, eps, (const TG*)gate, ldg, gate_col, act, (TO*)out, n_groups, size, gate_first, scale); \
+        if (vec && size <= 128) IB_GNV(TG, TO, 1);                                                                                  \
+        else if (vec && size <= 256) IB_GNV(TG, TO, 2);                                                                             \
+        else if (vec && size <= 512) IB_GNV(TG, TO, 4);                                                                             \
+        else if (vec) IB_GNV(TG, TO, 8);                                                                                            \
+        else if (wide) IB_LAUNCH((group_norm_gate_wide_kernel<TG, TO>), grid, 256, 0, o, w, eps, (const TG*)gate, ldg, gate_col, act, (TO*)out, n_groups, size, gate_first, scale); \
         else IB_LAUNCH((group_norm_gate_kernel<TG, TO>), grid, 256, 0, o, w, eps, (const TG*)gate, ldg, gate_col, act, (TO*)out, rows, n_groups, size, gate_first, scale);     \
     } while (0)
     if (!gate || gate_dtype == IB_F32) {
@@ -488,6 +577,7 @@ IB_EXPORT int ib_group_norm_gate(const float* o, const float* w, float eps, cons
         return ib::fail(IB_ERR_ARG, "ib_group_norm_gate: unknown gate dtype %d", gate_dtype);
     }
 #undef IB_GN
+#undef IB_GNV
     return ib::check_launch("ib_group_norm_gate");
 }
 

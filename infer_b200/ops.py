@@ -567,6 +567,27 @@ def route(logits: torch.Tensor, top: int, n_groups: int = 1, keep: int = 1, sum_
     return weights, chosen
 
 
+def route_rows(x: torch.Tensor, w: torch.Tensor, top: int, n_groups: int = 1, keep: int = 1, sum_eps: float = 0.0, want_chosen: bool = False,
+               sigmoid: bool = False, group_best: int = 1, renormalise: bool = True, mult: float = 1.0):
+    """``route`` of the logits x w^T, the product in the same kernel (x [T, W] and w [E, W] in one storage dtype, sums in
+    float32). None where the sizes are not the kernel's (more experts than it takes, rows that are no whole 16-byte pieces)."""
+    _check(x, "x")
+    _check(w, "w", x.dtype)
+    T, W = x.shape
+    E = w.shape[0]
+    if w.shape[1] != W:
+        raise KernelError(f"the router's matrix is {tuple(w.shape)}, the rows have {W} channels")
+    if W % 8 or E > int(_fn("mix", "ib_route_rows_max_experts", [])()) or (x.data_ptr() | w.data_ptr()) & 15:
+        return None
+    weights = torch.empty((T, E), dtype=torch.float32, device=x.device)
+    chosen = torch.empty((T, top), dtype=torch.int32, device=x.device) if want_chosen else None
+    f = _fn("mix", "ib_route_rows", [c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_float,
+                                     c_void_p, c_void_p, c_int, c_void_p])
+    _call(f, x.data_ptr(), w.data_ptr(), T, W, E, int(top), int(n_groups), int(keep), float(sum_eps), int(bool(sigmoid)), int(group_best),
+          int(bool(renormalise)), float(mult), weights.data_ptr(), _ptr(chosen), dtype_code(x.dtype), _stream())
+    return weights, chosen
+
+
 def rownorm_store(rows: torch.Tensor, col0: int, wq: Optional[torch.Tensor], wk: Optional[torch.Tensor], eps: float, step,
                   block_table: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, n_heads: int, n_kv: int,
                   head_dim: int, v_head_dim: int, write_cache: bool = True) -> torch.Tensor:

@@ -129,14 +129,14 @@ class RoutedExperts(FeedForward):
         return self._experts(weights, rows, residual)
 
     def _weights(self, x):
-        logits = self.router(x, out_dtype=torch.float32)
         if self.router_kind == "sigmoid":
-            weights, _ = ops.route_sigmoid(logits, self.correction, self.top, self.out_scale)
-        elif self.router_kind == "sigmoid_groups":
-            weights, _ = ops.route(logits, self.top, self.groups, self.keep, sigmoid=True, group_best=2, renormalise=False, mult=self.out_scale)
-        else:
-            weights, _ = ops.route(logits, self.top, self.groups, self.keep, self.sum_eps)
-        return weights
+            return ops.route_sigmoid(self.router(x, out_dtype=torch.float32), self.correction, self.top, self.out_scale)[0]
+        how = dict(sigmoid=True, group_best=2, renormalise=False, mult=self.out_scale) if self.router_kind == "sigmoid_groups" \
+            else dict(sum_eps=self.sum_eps)
+        got = ops.route_rows(x, self.router.weight, self.top, self.groups, self.keep, **how)      # the product in the same kernel
+        if got is None:
+            got = ops.route(self.router(x, out_dtype=torch.float32), self.top, self.groups, self.keep, **how)
+        return got[0]
 
     def _experts(self, weights, rows, residual):
         if self.expert_kind == "relu_squared":

@@ -174,7 +174,7 @@ def test_the_design_runs_on_its_own_kernels():
     H.run_trace(eng, [{"entries": [("x", ids[:139], [138])], "end": []}, {"entries": [("x", ids[139:], [0])], "end": ["x"]}])
     ran = {k: v - before.get(k, 0) for k, v in ops.LAUNCH_KINDS.items() if v != before.get(k, 0)}
     for kind in ("ib_state_scan", "ib_head_prepare", "ib_sum_norm", "ib_gate_mul", "ib_shift_mix", "ib_double_exp_decay",
-                 "ib_group_norm_gate", "ib_route", "ib_glu_act", "ib_relu_sq", "ib_silu_rows"):
+                 "ib_group_norm_gate", "ib_route_rows", "ib_glu_act", "ib_relu_sq", "ib_silu_rows"):
         assert ran.get(kind, 0) >= 2, (kind, ran)
     assert ran.get("ib_gemm_tc", 0) >= 1                     # the tensor-core product serves the prompt's matrices
     # keys and values of 64 and 128: the prompt's attention runs on the tensor-core kernel, with and without kept first

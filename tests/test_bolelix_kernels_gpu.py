@@ -174,6 +174,40 @@ def test_filter_steps_and_decays_over_steps(sizes):
         assert torch.equal(tails[0].cpu(), seqs[0][46 - taps + 1:, 3:3 + C])
 
 
+@pytest.mark.parametrize("taps", [1, 2, 3, 4, 5])
+def test_filter_over_prompt_portions_and_single_tokens_has_the_same_bits(taps):
+    """Long segments (several tokens a thread), a boundary inside a thread's tokens, and the same tokens in short steps."""
+    H, dv, N, G = 2, 12, 8, 1
+    C = H * dv + 2 * G * N
+    g = torch.Generator().manual_seed(taps)
+    n = (203, 130)
+    seqs = [torch.randn(m, C + H + 2, generator=g) for m in n]
+    fw, fb, dtb, al = torch.randn(C, taps, generator=g), torch.randn(C, generator=g), torch.randn(H, generator=g), torch.randn(H, generator=g)
+    d = lambda t: t.to(DEV).contiguous()
+
+    def run(cuts):
+        tails = torch.zeros(2, max(1, taps - 1), C, device=DEV) if taps > 1 else None
+        at, outs = [0, 0], [[], []]
+        for lens in cuts:
+            step = _Step(lens, list(at), [0, 1])
+            rows = d(torch.cat([s[a:a + m] for s, a, m in zip(seqs, at, lens)]))
+            out, g_col = ops.filter_prepare(rows, 0, d(fw.t()), d(fb), tails, C, d(dtb), d(al), step)
+            if tails is not None:
+                ops.tail_update(rows, 0, tails, step.seg_start, step.seg_slot)
+            out = out[:, :g_col + 3 * H].cpu()
+            outs[0].append(out[:lens[0]]), outs[1].append(out[lens[0]:])
+            at = [a + m for a, m in zip(at, lens)]
+        return [torch.cat(o) for o in outs]
+    whole, cut = run([[203, 130]]), run([[100, 65], [101, 1], [2, 64]])
+    for s in range(2):
+        assert torch.equal(whole[s], cut[s])
+        y = pb.silu(pb.causal_filter(seqs[s][:, :C].double(), fw, fb))
+        dt = pb.softplus(seqs[s][:, C:C + H].double() + dtb.double())
+        lng = -torch.exp(al.double()) * dt
+        want = torch.cat([y, torch.exp(lng), dt, lng], dim=1)
+        assert torch.allclose(whole[s].double(), want, rtol=2e-5, atol=2e-5)
+
+
 SCAN_SIZES = [(2, 2, 16, 32), (4, 2, 40, 20), (3, 1, 5, 9), (2, 1, 128, 64), (4, 4, 8, 4), (2, 2, 160, 128), (1, 1, 33, 3), (6, 3, 64, 24)]
 
 
@@ -366,3 +400,22 @@ def test_normalised_read_out_with_head_norm_and_gate(H, dv, dtype):
     x = mult * o.double().view(T, H, dv) / (torch.maximum((mult * den.double()).abs(), low[:, 2:].double()) + floor)[:, :, None]
     want = pb.rms(x, eps).view(T, -1) * w.double() * torch.sigmoid(z[:, 4:].double())
     assert torch.allclose(got.double().cpu(), want, **_tol(dtype))
+
+
+# ----------------------------------------------------------------------------------------------- the router
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16], ids=["f32", "bf16"])
+@pytest.mark.parametrize("E,top,width", [(8, 2, 1536), (4, 4, 8), (9, 1, 264), (16, 4, 40), (33, 3, 512), (64, 6, 1000), (3, 2, 72)])
+def test_router_with_its_product(E, top, width, dtype):
+    g = torch.Generator().manual_seed(E)
+    x, w = torch.randn(37, width, generator=g).to(dtype), (torch.randn(E, width, generator=g) * width ** -0.5 * 2).to(dtype)
+    weights, chosen = ops.route_rows(x.to(DEV), w.to(DEV), top, want_chosen=True)
+    z = x.double() @ w.double().T
+    want, ww, gap = pb.route_top(z, top)
+    clear = gap > 1e-4
+    assert int(clear.sum()) >= 30
+    assert torch.equal(chosen.cpu().long()[clear], want[clear])
+    full = torch.zeros(37, E, dtype=F).scatter_(1, want, ww)
+    assert torch.allclose(weights.double().cpu()[clear], full[clear], rtol=1e-4, atol=1e-6)
+    assert torch.equal(ops.route_rows(x[5:6].to(DEV).contiguous(), w.to(DEV), top)[0][0], weights[5])      # whatever else is in the step
+    assert ops.route_rows(torch.zeros(2, 12, device=DEV), torch.zeros(4, 12, device=DEV), 1) is None       # no whole pieces: another path

@@ -173,7 +173,7 @@ def test_the_design_runs_on_its_own_kernels():
     before = dict(ops.LAUNCH_KINDS)
     H.run_trace(eng, [{"entries": [("x", ids[:139], [138])], "end": []}, {"entries": [("x", ids[139:], [0])], "end": ["x"]}])
     ran = {k: v - before.get(k, 0) for k, v in ops.LAUNCH_KINDS.items() if v != before.get(k, 0)}
-    for kind in ("ib_state_scan", "ib_delta_prepare", "ib_decay_gates", "ib_rownorm_store", "ib_route", "ib_glu_act", "ib_norm_add",
+    for kind in ("ib_state_scan", "ib_delta_prepare", "ib_decay_gates", "ib_rownorm_store", "ib_route_rows", "ib_glu_act", "ib_norm_add",
                  "ib_dual_norm_sum", "ib_head_norm_gate"):
         assert ran.get(kind, 0) >= 2, (kind, ran)
     assert ran.get("ib_gemm_tc", 0) >= 1                     # the tensor-core product serves the prompt's matrices

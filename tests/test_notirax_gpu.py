@@ -173,7 +173,7 @@ def test_the_design_runs_on_its_own_kernels():
     before = dict(ops.LAUNCH_KINDS)
     H.run_trace(eng, [{"entries": [("x", ids[:139], [138])], "end": []}, {"entries": [("x", ids[139:], [0])], "end": ["x"]}])
     ran = {k: v - before.get(k, 0) for k, v in ops.LAUNCH_KINDS.items() if v != before.get(k, 0)}
-    for kind in ("ib_embedding_sinusoid", "ib_stream_link", "ib_delta_prepare", "ib_state_scan", "ib_group_norm_gate", "ib_route", "ib_glu_act"):
+    for kind in ("ib_embedding_sinusoid", "ib_stream_link", "ib_delta_prepare", "ib_state_scan", "ib_group_norm_gate", "ib_route_rows", "ib_glu_act"):
         assert ran.get(kind, 0) >= 2, (kind, ran)
     assert ran.get("ib_gemm_tc", 0) >= 1                     # the tensor-core product serves the prompt's matrices
     # keys and values of 64 and 128: the prompt's attention runs on the tensor-core kernels, every decoded token's on the
