@@ -218,20 +218,22 @@ chunk_scan_kernel(const float* __restrict__ rows, int64_t ld, int q_col, int k_c
 #pragma unroll
                 for (int m = 0; m < MT; m++)
                     ldm4t(a[m], &sm.k[buf][kk * 16 + (lane >> 4) * 8 + (lane & 7)][d0 + 16 * m + ((lane >> 3) & 1) * 8]);
+                uint32_t bh[NT / 2][4], bl[NT / 2][4];        // tokens x two column tiles each
 #pragma unroll
                 for (int n2 = 0; n2 < NT / 2; n2++) {
-                    uint32_t bh[4], bl[4];                    // tokens x two column tiles
                     const int row = kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), col = 16 * n2 + (lane >> 4) * 8;
-                    ldm4t(bh, &sm.wh[buf][row][col]);
-                    ldm4t(bl, &sm.wl[buf][row][col]);
-#pragma unroll
-                    for (int m = 0; m < MT; m++) {
-                        mma(S[m][2 * n2], a[m], bh[0], bh[1]);
-                        mma(S[m][2 * n2 + 1], a[m], bh[2], bh[3]);
-                        mma(S[m][2 * n2], a[m], bl[0], bl[1]);
-                        mma(S[m][2 * n2 + 1], a[m], bl[2], bl[3]);
-                    }
+                    ldm4t(bh[n2], &sm.wh[buf][row][col]);
+                    ldm4t(bl[n2], &sm.wl[buf][row][col]);
                 }
+                // (products that add to one fragment stand as far apart as there are fragments)
+#pragma unroll
+                for (int m = 0; m < MT; m++)
+#pragma unroll
+                    for (int n = 0; n < NT; n++) mma(S[m][n], a[m], bh[n / 2][(n & 1) * 2], bh[n / 2][(n & 1) * 2 + 1]);
+#pragma unroll
+                for (int m = 0; m < MT; m++)
+#pragma unroll
+                    for (int n = 0; n < NT; n++) mma(S[m][n], a[m], bl[n / 2][(n & 1) * 2], bl[n / 2][(n & 1) * 2 + 1]);
             }
             if (c + 1 < n_chunks) {
                 leave_state(buf ^ 1);
@@ -261,17 +263,17 @@ chunk_scan_kernel(const float* __restrict__ rows, int64_t ld, int q_col, int k_c
                 for (int e = 0; e < 4; e++) o[n][e] = 0.0f;
 #pragma unroll
             for (int kk = 0; kk < KT; kk++) {
+                uint32_t bh[NT / 2][4], bl[NT / 2][4];
 #pragma unroll
                 for (int n2 = 0; n2 < NT / 2; n2++) {
-                    uint32_t bh[4], bl[4];
                     const int row = kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), col = 16 * n2 + (lane >> 4) * 8;
-                    ldm4t(bh, &sm.sh[buf][row][col]);
-                    ldm4t(bl, &sm.sl[buf][row][col]);
-                    mma(o[2 * n2], q[kk], bh[0], bh[1]);
-                    mma(o[2 * n2 + 1], q[kk], bh[2], bh[3]);
-                    mma(o[2 * n2], q[kk], bl[0], bl[1]);
-                    mma(o[2 * n2 + 1], q[kk], bl[2], bl[3]);
+                    ldm4t(bh[n2], &sm.sh[buf][row][col]);
+                    ldm4t(bl[n2], &sm.sl[buf][row][col]);
                 }
+#pragma unroll
+                for (int n = 0; n < NT; n++) mma(o[n], q[kk], bh[n / 2][(n & 1) * 2], bh[n / 2][(n & 1) * 2 + 1]);
+#pragma unroll
+                for (int n = 0; n < NT; n++) mma(o[n], q[kk], bl[n / 2][(n & 1) * 2], bl[n / 2][(n & 1) * 2 + 1]);
             }
             const int ra = r0 + fr, rb = ra + 8;
             const float ha = sm.ch[buf][ra], la = sm.cl[buf][ra], hb = sm.ch[buf][rb], lb = sm.cl[buf][rb];
@@ -282,18 +284,22 @@ chunk_scan_kernel(const float* __restrict__ rows, int64_t ld, int q_col, int k_c
 #pragma unroll
             for (int j = 0; j < L / 16; j++) {
                 if (j > gw) break;
-                float s[2][4];
+                float s[2][4], s2[2][4];                      // (even and odd steps over the channels)
 #pragma unroll
                 for (int i = 0; i < 2; i++)
 #pragma unroll
-                    for (int e = 0; e < 4; e++) s[i][e] = 0.0f;
+                    for (int e = 0; e < 4; e++) s[i][e] = s2[i][e] = 0.0f;
 #pragma unroll
                 for (int kk = 0; kk < KT; kk++) {
                     uint32_t kb[4];                           // keys 16 j + (0..7 | 8..15), channels in two halves
                     ldm4(kb, &sm.k[buf][16 * j + (lane >> 4) * 8 + (lane & 7)][kk * 16 + ((lane >> 3) & 1) * 8]);
-                    mma(s[0], q[kk], kb[0], kb[1]);
-                    mma(s[1], q[kk], kb[2], kb[3]);
+                    mma((kk & 1) ? s2[0] : s[0], q[kk], kb[0], kb[1]);
+                    mma((kk & 1) ? s2[1] : s[1], q[kk], kb[2], kb[3]);
                 }
+#pragma unroll
+                for (int i = 0; i < 2; i++)
+#pragma unroll
+                    for (int e = 0; e < 4; e++) s[i][e] += s2[i][e];
                 uint32_t ph[4], pl[4];
 #pragma unroll
                 for (int i = 0; i < 2; i++) {
@@ -307,15 +313,14 @@ chunk_scan_kernel(const float* __restrict__ rows, int64_t ld, int q_col, int k_c
                     split2(p0, p1, ph[2 * i], pl[2 * i]);
                     split2(p2, p3, ph[2 * i + 1], pl[2 * i + 1]);
                 }
+                uint32_t vb[NT / 2][4];
 #pragma unroll
-                for (int n2 = 0; n2 < NT / 2; n2++) {
-                    uint32_t vb[4];
-                    ldm4t(vb, &sm.v[buf][16 * j + ((lane >> 3) & 1) * 8 + (lane & 7)][16 * n2 + (lane >> 4) * 8]);
-                    mma(o[2 * n2], ph, vb[0], vb[1]);
-                    mma(o[2 * n2 + 1], ph, vb[2], vb[3]);
-                    mma(o[2 * n2], pl, vb[0], vb[1]);
-                    mma(o[2 * n2 + 1], pl, vb[2], vb[3]);
-                }
+                for (int n2 = 0; n2 < NT / 2; n2++)
+                    ldm4t(vb[n2], &sm.v[buf][16 * j + ((lane >> 3) & 1) * 8 + (lane & 7)][16 * n2 + (lane >> 4) * 8]);
+#pragma unroll
+                for (int n = 0; n < NT; n++) mma(o[n], ph, vb[n / 2][(n & 1) * 2], vb[n / 2][(n & 1) * 2 + 1]);
+#pragma unroll
+                for (int n = 0; n < NT; n++) mma(o[n], pl, vb[n / 2][(n & 1) * 2], vb[n / 2][(n & 1) * 2 + 1]);
             }
 #pragma unroll
             for (int half = 0; half < 2; half++) {

@@ -261,15 +261,22 @@ filter_prepare_tokens_kernel(const float* __restrict__ rows, int64_t ld, int col
 //   i = cap tanh((raw[i_col + h] + i_bias[h]) / cap),   f = log sigmoid(cap tanh((raw[f_col + h] + f_bias[h]) / cap))
 //   m <- max(f + m, i)   (m kept per request and head in `state` [slots, H], zero for a new request)
 //   out rows (ldo): [keep = exp(f + m_before - m) (H) | write = exp(i - m) (H) | floor = exp(-m) (H) | ln keep (H)]
-// The gates and the exponentials are computed in parallel over a tile of tokens; the running maximum walks the tile in
-// one thread, an addition and a maximum a token, so that it does not depend on where a prompt was cut.
-constexpr int GATE_TILE = 512;
+// The gates and the exponentials are computed in parallel over a tile of tokens. The running maximum walks the tile in one
+// thread, an addition and a maximum a token, so that it does not depend on where a prompt was cut. With `blocks` (where its
+// last bits may) a tile of n tokens is cut into blocks of GATE_BLOCK: what a block makes of the maximum in front of it is
+// max(a + m, b), and a thread per block finds a (its sum of f) and b; a walk over the blocks gives the maximum in front of
+// each, and the threads walk their blocks again from there.
+constexpr int GATE_TILE = 2048, GATE_BLOCK = 32;
 
 __global__ void __launch_bounds__(512)
 memory_gates_kernel(const float* __restrict__ rows, int64_t ld, int i_col, int f_col, const float* __restrict__ i_bias,
                     const float* __restrict__ f_bias, float cap, float* __restrict__ state, const int* __restrict__ seg_start,
-                    const int* __restrict__ seg_slot, float* __restrict__ out, int64_t ldo, int n_heads, int write_state) {
-    __shared__ __align__(16) float gi[GATE_TILE + 4], gf[GATE_TILE + 4], gm[GATE_TILE + 4];
+                    const int* __restrict__ seg_slot, float* __restrict__ out, int64_t ldo, int n_heads, int write_state, int blocks) {
+    // (a block's tokens start one place further on than the last block's: threads that walk neighbouring blocks use
+    // different banks)
+    __shared__ __align__(16) float gi[GATE_TILE + GATE_TILE / GATE_BLOCK + 8], gf[GATE_TILE + GATE_TILE / GATE_BLOCK + 8];
+    __shared__ __align__(16) float gm[GATE_TILE + GATE_TILE / GATE_BLOCK + 8];
+    __shared__ float ba[GATE_TILE / GATE_BLOCK], bb[GATE_TILE / GATE_BLOCK], bm[GATE_TILE / GATE_BLOCK + 1];
     ib::pdl_launch_dependents();
     ib::pdl_wait();
     const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
@@ -278,16 +285,48 @@ memory_gates_kernel(const float* __restrict__ rows, int64_t ld, int i_col, int f
     float* kept = state + int64_t(seg_slot[s]) * n_heads + h;
     const float bi = i_bias[h], bf = f_bias[h];
     float m = *kept;
+    const int pad = blocks ? 1 : 0;
+    auto at = [&](int c) { return c + pad * (c / GATE_BLOCK); };
     for (int c0 = 0; c0 < len; c0 += GATE_TILE) {
         const int n = min(GATE_TILE, len - c0);
         for (int c = tid; c < n; c += blockDim.x) {
             const float* r = rows + (t0 + c0 + c) * ld;
-            gi[c] = cap * tanhf((r[i_col + h] + bi) / cap);
-            gf[c] = log_sigmoid_(cap * tanhf((r[f_col + h] + bf) / cap));
+            gi[at(c)] = cap * tanhf((r[i_col + h] + bi) / cap);
+            gf[at(c)] = log_sigmoid_(cap * tanhf((r[f_col + h] + bf) / cap));
         }
         __syncthreads();
-        if (tid == 0) {
-            // gm[c] is the maximum before token c, gm[n] the one after the tile
+        // gm[at(c)] is the maximum before token c; bm[last] the one after the tile
+        const int n_blocks = (n + GATE_BLOCK - 1) / GATE_BLOCK;
+        if (blocks) {
+            if (tid < n_blocks) {
+                const int c1 = min(n, (tid + 1) * GATE_BLOCK);
+                float a = 0.0f, b = -INFINITY;
+                for (int c = tid * GATE_BLOCK; c < c1; c++) {
+                    const float f = gf[at(c)];
+                    a += f;
+                    b = fmaxf(f + b, gi[at(c)]);
+                }
+                ba[tid] = a;
+                bb[tid] = b;
+            }
+            __syncthreads();
+            if (tid == 0) {
+                for (int k = 0; k < n_blocks; k++) {
+                    bm[k] = m;
+                    m = fmaxf(ba[k] + m, bb[k]);
+                }
+            }
+            __syncthreads();
+            if (tid < n_blocks) {
+                const int c1 = min(n, (tid + 1) * GATE_BLOCK);
+                float mm = bm[tid];
+                for (int c = tid * GATE_BLOCK; c < c1; c++) {
+                    gm[at(c)] = mm;
+                    mm = fmaxf(gf[at(c)] + mm, gi[at(c)]);
+                }
+                if (tid == n_blocks - 1) bm[n_blocks] = mm;
+            }
+        } else if (tid == 0) {
             int c = 0;
             float4 i_next = load4(gi), f_next = load4(gf);   // (four tokens ahead of the walk)
             for (; c + 4 <= n; c += 4) {
@@ -309,19 +348,20 @@ memory_gates_kernel(const float* __restrict__ rows, int64_t ld, int i_col, int f
                 gm[c] = m;
                 m = fmaxf(gf[c] + m, gi[c]);
             }
-            gm[n] = m;
+            bm[n_blocks] = m;
         }
         __syncthreads();
         for (int c = tid; c < n; c += blockDim.x) {
             float* o = out + (t0 + c0 + c) * ldo;
-            const float now = gm[c + 1];
-            const float lnk = gf[c] + gm[c] - now;
+            const float f = gf[at(c)], i = gi[at(c)], before = gm[at(c)];
+            const float now = fmaxf(f + before, i);
+            const float lnk = f + before - now;
             o[h] = expf(lnk);
-            o[n_heads + h] = expf(gi[c] - now);
+            o[n_heads + h] = expf(i - now);
             o[2 * n_heads + h] = expf(-now);
             o[3 * n_heads + h] = lnk;
         }
-        m = gm[n];
+        m = bm[n_blocks];
         __syncthreads();
     }
     if (write_state && tid == 0) *kept = m;
@@ -385,12 +425,12 @@ IB_EXPORT int ib_filter_prepare(const float* rows, int64_t ld, int col0, int cha
 
 IB_EXPORT int ib_memory_gates(const float* rows, int64_t ld, int i_col, int f_col, const float* i_bias, const float* f_bias, float cap,
                               float* state, const int* seg_start, const int* seg_slot, float* out, int64_t ldo, int n_segments,
-                              int n_heads, int write_state, int max_len, cudaStream_t stream) {
+                              int n_heads, int write_state, int max_len, int blocks, cudaStream_t stream) {
     if (n_segments <= 0) return IB_OK;
     if (n_heads <= 0 || n_heads > 65535 || !(cap > 0.0f) || ldo < 4 * int64_t(n_heads))
         return ib::fail(IB_ERR_ARG, "ib_memory_gates: %d heads, a cap of %f", n_heads, double(cap));
     // (the number of threads changes nothing but how many tokens of a tile are formed at a time)
     IB_LAUNCH(memory_gates_kernel, (dim3{unsigned(n_segments), unsigned(n_heads), 1u}), max_len > 32 ? 512 : 32, 0, rows, ld, i_col, f_col, i_bias, f_bias, cap,
-              state, seg_start, seg_slot, out, ldo, n_heads, write_state);
+              state, seg_start, seg_slot, out, ldo, n_heads, write_state, blocks && max_len > 2 * GATE_BLOCK);
     return ib::check_launch("ib_memory_gates");
 }

@@ -310,25 +310,23 @@ route_rows_kernel(const T* __restrict__ x, const T* __restrict__ w, int64_t n_to
     float acc[EB];
 #pragma unroll
     for (int e = 0; e < EB; e++) acc[e] = 0.0f;
+    // no branch around a row of the matrix (the last one stands in for those beyond it): all loads of a pass go out together
+#pragma unroll 2
     for (int i = lane * 8; i < width; i += 256) {
         float xv[8];
         load8<T>(x + t * width + i, xv);
 #pragma unroll
         for (int e = 0; e < EB; e++) {
-            if (e < n_experts) {
-                float wv[8];
-                load8<T>(w + int64_t(e) * width + i, wv);
+            float wv[8];
+            load8<T>(w + int64_t(min(e, n_experts - 1)) * width + i, wv);
 #pragma unroll
-                for (int j = 0; j < 8; j++) acc[e] = fmaf(xv[j], wv[j], acc[e]);
-            }
+            for (int j = 0; j < 8; j++) acc[e] = fmaf(xv[j], wv[j], acc[e]);
         }
     }
 #pragma unroll
     for (int e = 0; e < EB; e++) {
-        if (e < n_experts) {
-            const float z = ib::warp_sum(acc[e]);
-            if (lane == e % 32) s[e] = z;
-        }
+        const float z = ib::warp_sum(acc[e]);
+        if (lane == e % 32 && e < n_experts) s[e] = z;
     }
     __syncwarp();
     route_token(s, s, s + n_experts, t, lane, n_experts, top, n_groups, keep, sum_eps, sigmoid, group_best, renormalise, mult, weights, chosen);

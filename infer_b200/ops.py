@@ -1563,11 +1563,12 @@ def filter_prepare(rows: torch.Tensor, col0: int, filt_w: torch.Tensor, filt_b: 
 
 
 def memory_gates(rows: torch.Tensor, i_col: int, f_col: int, i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float, state: torch.Tensor,
-                 step, write_state: bool = True) -> torch.Tensor:
+                 step, write_state: bool = True, blocks: bool = False) -> torch.Tensor:
     """Gates of a matrix memory over the tokens of every segment in order, from float32 projected rows: with
     i = cap tanh((raw_i + i_bias) / cap) and f = log sigmoid(cap tanh((raw_f + f_bias) / cap)) per head, m <- max(f + m, i)
     (kept in ``state`` float32 [slots, heads]). Returns float32 [T, exp(f + m_before - m) | exp(i - m) | exp(-m) | f + m_before - m],
-    heads each."""
+    heads each. ``blocks``: long segments may find m a block of tokens at a time (its last bits may then depend on where a
+    prompt was cut)."""
     _check(rows, "rows", torch.float32)
     T, ld = rows.shape
     H = i_bias.numel()
@@ -1578,9 +1579,9 @@ def memory_gates(rows: torch.Tensor, i_col: int, f_col: int, i_bias: torch.Tenso
         raise KernelError("memory_gates: columns lie outside the rows")
     out = torch.empty((T, 4 * H), dtype=torch.float32, device=rows.device)
     f = _fn("memory", "ib_memory_gates", [c_void_p, c_int64, c_int, c_int, c_void_p, c_void_p, c_float] + [c_void_p] * 4 +
-            [c_int64, c_int, c_int, c_int, c_int, c_void_p])
+            [c_int64, c_int, c_int, c_int, c_int, c_int, c_void_p])
     _call(f, rows.data_ptr(), ld, int(i_col), int(f_col), i_bias.data_ptr(), f_bias.data_ptr(), float(cap), state.data_ptr(),
-          step.seg_start.data_ptr(), step.seg_slot.data_ptr(), out.data_ptr(), 4 * H, step.seg_slot.numel(), H, int(write_state), int(step.max_q_len), _stream())
+          step.seg_start.data_ptr(), step.seg_slot.data_ptr(), out.data_ptr(), 4 * H, step.seg_slot.numel(), H, int(write_state), int(step.max_q_len), int(bool(blocks)), _stream())
     return out
 
 

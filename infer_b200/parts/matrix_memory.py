@@ -97,7 +97,8 @@ class MatrixMemory(Mixer):
         H, nq, nv = self.n_heads, self.n_heads * self.dim, self.n_heads * self.v_dim
         rows, c0 = own_or_projected(self, x, self.proj, torch.float32)
         gate_col = c0 + 2 * nq + nv
-        gates = ops.memory_gates(rows, gate_col + nv, gate_col + nv + H, self.input_b, self.forget_b, self.cap, cache["m"], step, write_cache)
+        gates = ops.memory_gates(rows, gate_col + nv, gate_col + nv + H, self.input_b, self.forget_b, self.cap, cache["m"], step, write_cache,
+                                 blocks=self.rt.dtype == torch.bfloat16)
         o, den = ops.step_scan(rows, c0, c0 + nq, c0 + 2 * nq, gates, 0, H, 3 * H, cache["S"], step, H, 1, self.dim, self.v_dim, write_cache,
                                ones_state=cache["n"], chunked=self.rt.dtype == torch.bfloat16)
         # (the read-outs are linear in q: its constant is applied to them)

@@ -349,7 +349,7 @@ def test_memory_gates_over_steps(H, cap):
     """The running maximum over unequal segments, cuttings bit-equal; the second sequence is longer than a tile."""
     g = torch.Generator().manual_seed(H)
     bi, bf = torch.randn(H, generator=g), 2.0 + torch.randn(H, generator=g)
-    seqs = {0: 6 * torch.randn(46, 2 + 2 * H, generator=g), 2: 6 * torch.randn(1225, 2 + 2 * H, generator=g)}
+    seqs = {0: 6 * torch.randn(46, 2 + 2 * H, generator=g), 2: 6 * torch.randn(2225, 2 + 2 * H, generator=g)}
     ref = {}
     for s, r in seqs.items():
         i, f = pb.memory_gates(r[:, 2:2 + H].double() + bi.double(), r[:, 2 + H:].double() + bf.double(), cap)
@@ -361,7 +361,7 @@ def test_memory_gates_over_steps(H, cap):
         ref[s] = torch.stack(rows)
     d = lambda t: t.to(DEV).contiguous()
 
-    def run(all_lens):
+    def run(all_lens, blocks=False):
         state = torch.full((3, H), float("nan"), device=DEV)
         state[0].zero_(), state[2].zero_()
         at, outs = {0: 0, 2: 0}, {0: [], 2: []}
@@ -369,7 +369,7 @@ def test_memory_gates_over_steps(H, cap):
             step = _Step(lens, [at[0], at[2]], [0, 2])
             rows = d(torch.cat([seqs[s][at[s]:at[s] + m] for s, m in zip((0, 2), lens)]))
             step.max_q_len = max(lens)
-            got = ops.memory_gates(rows, 2, 2 + H, d(bi), d(bf), cap, state, step).cpu()
+            got = ops.memory_gates(rows, 2, 2 + H, d(bi), d(bf), cap, state, step, blocks=blocks).cpu()
             assert torch.allclose(got[:, 3 * H:].exp(), got[:, :H], rtol=1e-6)
             got = got[:, :3 * H]
             outs[0].append(got[:lens[0]]), outs[2].append(got[lens[0]:])
@@ -377,11 +377,14 @@ def test_memory_gates_over_steps(H, cap):
                 at[s] += m
         assert bool(torch.isnan(state[1]).all())
         return {s: torch.cat(o) for s, o in outs.items()}
-    a = run([[1, 2], [2, 1], [17, 9], [1, 1], [25, 1212]])
-    b = run([[45, 1224], [1, 1]])
+    a = run([[1, 2], [2, 1], [17, 9], [1, 1], [25, 2212]])
+    b = run([[45, 2224], [1, 1]])
+    c, e = run([[45, 2224], [1, 1]], True), run([[1, 3], [33, 65], [12, 2157]], True)
     for s in (0, 2):
         assert torch.allclose(a[s].double(), ref[s], rtol=3e-5, atol=1e-6)
         assert torch.equal(a[s], b[s])
+        for x in (c, e):                                     # a block of tokens at a time: up to rounding
+            assert torch.allclose(x[s].double(), ref[s], rtol=3e-5, atol=1e-6)
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16], ids=["f32", "bf16"])
