@@ -295,24 +295,24 @@ route_kernel(const float* __restrict__ logits, int64_t n_tokens, int n_experts, 
 }
 
 // The same with the router's product in front of it: logits = W x in float, rows and matrix in storage T (widths of whole
-// 16-byte pieces, up to EB experts). One warp per token, its lanes along the row; a token's sums do not depend on the others.
+// 16-byte pieces, up to EB experts). One CTA of four warps per token, each with a share of the row; the shares' sums meet in
+// a fixed order, so that a token's logits do not depend on what else is in the step.
 template <typename T, int EB>
 __global__ void __launch_bounds__(128)
-route_rows_kernel(const T* __restrict__ x, const T* __restrict__ w, int64_t n_tokens, int width, int n_experts, int top, int n_groups,
+route_rows_kernel(const T* __restrict__ x, const T* __restrict__ w, int width, int n_experts, int top, int n_groups,
                   int keep, float sum_eps, int sigmoid, int group_best, int renormalise, float mult, float* __restrict__ weights,
                   int* __restrict__ chosen) {
     ib::pdl_wait();
-    extern __shared__ float sm[];
+    extern __shared__ float sm[];                            // [experts + groups] of the routing, [4][EB] shares
+    float* part = sm + n_experts + n_groups;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int64_t t = int64_t(blockIdx.x) * (blockDim.x >> 5) + warp;
-    if (t >= n_tokens) return;
-    float* s = sm + warp * (n_experts + n_groups);
+    const int64_t t = blockIdx.x;
     float acc[EB];
 #pragma unroll
     for (int e = 0; e < EB; e++) acc[e] = 0.0f;
     // no branch around a row of the matrix (the last one stands in for those beyond it): all loads of a pass go out together
 #pragma unroll 2
-    for (int i = lane * 8; i < width; i += 256) {
+    for (int i = threadIdx.x * 8; i < width; i += 1024) {
         float xv[8];
         load8<T>(x + t * width + i, xv);
 #pragma unroll
@@ -326,10 +326,13 @@ route_rows_kernel(const T* __restrict__ x, const T* __restrict__ w, int64_t n_to
 #pragma unroll
     for (int e = 0; e < EB; e++) {
         const float z = ib::warp_sum(acc[e]);
-        if (lane == e % 32 && e < n_experts) s[e] = z;
+        if (lane == e % 32) part[warp * EB + e] = z;
     }
+    __syncthreads();
+    if (warp > 0) return;
+    for (int e = lane; e < n_experts; e += 32) sm[e] = (part[e] + part[EB + e]) + (part[2 * EB + e] + part[3 * EB + e]);
     __syncwarp();
-    route_token(s, s, s + n_experts, t, lane, n_experts, top, n_groups, keep, sum_eps, sigmoid, group_best, renormalise, mult, weights, chosen);
+    route_token(sm, sm, sm + n_experts, t, lane, n_experts, top, n_groups, keep, sum_eps, sigmoid, group_best, renormalise, mult, weights, chosen);
 }
 
 // ------------------------------------------------------------------------------------------------
@@ -423,67 +426,79 @@ split_attention_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
         const int gq = i / d, e = i - gq * d;
         qs[gq * dq + e] = ib::to_f32(q[(t * n_heads + h0 + gq) * d + e]);
     }
-    __syncthreads();
     const int* table = block_table + int64_t(sg) * max_blocks;
     const int key = base + tid;
     const bool valid = key <= pos && (key >= lo || key < keep_end);
     // a key in the gap between the kept keys and the window takes the row of the chunk's first visible key (weight 0)
     const int first_seen = base < keep_end ? base : max(lo, base);
     const bool in_gap = !valid && key > first_seen && key < lo;
+    const int j0 = first_seen - base, j1 = (ci < nk ? min(keep_end - 1, base + KC - 1) : min(pos, base + KC - 1)) - base;
     float acc[GB];
 #pragma unroll
     for (int gq = 0; gq < GB; gq++) acc[gq] = 0.0f;
     bool have = false;
-    if (in_gap) {
-        const int page = table[first_seen / page_size];
-        rowoff[tid] = (page < 0 || page >= n_pages) ? 0 : (int64_t(page) * n_kv + g) * page_size + first_seen % page_size;
-    } else if (valid) {
-        const int page = table[key / page_size];
-        if (page < 0 || page >= n_pages) {
-            if (status) atomicExch(status, 3);
-            rowoff[tid] = 0;
-        } else {
-            have = true;
-            const int64_t row = (int64_t(page) * n_kv + g) * page_size + key % page_size;
-            rowoff[tid] = row;
-            const T* kr = k_cache + row * d;
-            if (vec) {
-                // four 16-byte loads of the row are in flight together (a thread's row is its own: nothing is shared)
-                for (int e0 = 0; e0 < d; e0 += 32) {
-                    float kv[4][8];
+    int64_t row = 0;
+    if (valid || in_gap) {
+        const int k_at = valid ? key : first_seen;
+        const int page = table[k_at / page_size];
+        if (page >= 0 && page < n_pages) {
+            row = (int64_t(page) * n_kv + g) * page_size + k_at % page_size;
+            have = valid;
+        } else if (valid && status) {
+            atomicExch(status, 3);
+        }
+    }
+    rowoff[tid] = row;
+    __syncthreads();                                    // queries and row places have arrived
+    T* vt = reinterpret_cast<T*>(rowoff + KC);          // vec_v 1: [VT][dv]; 2: [KC][dv]
+    if (vec_v == 2) {
+        // all value rows are on their way while the scores are computed
+        constexpr int PER = 16 / int(sizeof(T));
+        const int per_row = dv / PER, n16 = (j1 - j0 + 1) * per_row;
+        for (int i = tid; i < n16; i += KC) {
+            const int jj = j0 + i / per_row, e = (i % per_row) * PER;
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(uint32_t(__cvta_generic_to_shared(vt + jj * dv + e))),
+                         "l"(v_cache + rowoff[jj] * dv + e) : "memory");
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    }
+    if (have) {
+        const T* kr = k_cache + row * d;
+        if (vec) {
+            // eight 16-byte loads of the row are in flight together (a thread's row is its own: nothing is shared)
+            constexpr int AHEAD = GB >= 16 ? 4 : 8;
+            for (int e0 = 0; e0 < d; e0 += 8 * AHEAD) {
+                float kv[AHEAD][8];
 #pragma unroll
-                    for (int b4 = 0; b4 < 4; b4++) {
-                        if (e0 + 8 * b4 < d) load8<T>(kr + e0 + 8 * b4, kv[b4]);
-                    }
+                for (int b4 = 0; b4 < AHEAD; b4++) {
+                    if (e0 + 8 * b4 < d) load8<T>(kr + e0 + 8 * b4, kv[b4]);
+                }
 #pragma unroll
-                    for (int b4 = 0; b4 < 4; b4++) {
-                        const int e = e0 + 8 * b4;
-                        if (e < d) {
+                for (int b4 = 0; b4 < AHEAD; b4++) {
+                    const int e = e0 + 8 * b4;
+                    if (e < d) {
 #pragma unroll
-                            for (int gq = 0; gq < GB; gq++) {
-                                if (gq < group) {
-                                    const float4 a = *reinterpret_cast<const float4*>(qs + gq * dq + e);
-                                    const float4 b = *reinterpret_cast<const float4*>(qs + gq * dq + e + 4);
-                                    float x = acc[gq];
-                                    x = fmaf(a.x, kv[b4][0], x); x = fmaf(a.y, kv[b4][1], x); x = fmaf(a.z, kv[b4][2], x); x = fmaf(a.w, kv[b4][3], x);
-                                    x = fmaf(b.x, kv[b4][4], x); x = fmaf(b.y, kv[b4][5], x); x = fmaf(b.z, kv[b4][6], x); x = fmaf(b.w, kv[b4][7], x);
-                                    acc[gq] = x;
-                                }
+                        for (int gq = 0; gq < GB; gq++) {
+                            if (gq < group) {
+                                const float4 a = *reinterpret_cast<const float4*>(qs + gq * dq + e);
+                                const float4 b = *reinterpret_cast<const float4*>(qs + gq * dq + e + 4);
+                                float x = acc[gq];
+                                x = fmaf(a.x, kv[b4][0], x); x = fmaf(a.y, kv[b4][1], x); x = fmaf(a.z, kv[b4][2], x); x = fmaf(a.w, kv[b4][3], x);
+                                x = fmaf(b.x, kv[b4][4], x); x = fmaf(b.y, kv[b4][5], x); x = fmaf(b.z, kv[b4][6], x); x = fmaf(b.w, kv[b4][7], x);
+                                acc[gq] = x;
                             }
                         }
                     }
                 }
-            } else {
-                for (int e = 0; e < d; e++) {
-                    const float kv = ib::to_f32(kr[e]);
+            }
+        } else {
+            for (int e = 0; e < d; e++) {
+                const float kv = ib::to_f32(kr[e]);
 #pragma unroll
-                    for (int gq = 0; gq < GB; gq++)
-                        if (gq < group) acc[gq] = fmaf(qs[gq * dq + e], kv, acc[gq]);
-                }
+                for (int gq = 0; gq < GB; gq++)
+                    if (gq < group) acc[gq] = fmaf(qs[gq * dq + e], kv, acc[gq]);
             }
         }
-    } else {
-        rowoff[tid] = 0;
     }
 #pragma unroll
     for (int gq = 0; gq < GB; gq++) {
@@ -513,25 +528,29 @@ split_attention_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
         if (lane == 0) { ml[2 * gq] = m; ml[2 * gq + 1] = l; }
     }
     __syncthreads();
-    const int j0 = first_seen - base, j1 = (ci < nk ? min(keep_end - 1, base + KC - 1) : min(pos, base + KC - 1)) - base;
     if (vec_v) {
-        // Value rows reach shared memory VT keys at a time, by 16-byte loads that all threads issue together; then a
-        // thread per channel adds them in ascending key order (the same order as the loop below).
-        T* vt = reinterpret_cast<T*>(rowoff + KC);           // [VT][dv]
+        // Value rows reach shared memory, all at once (requested above) or VT keys at a time by 16-byte loads that all threads
+        // issue together; then a thread per channel adds them in ascending key order (the same order as the loop below).
         constexpr int PER = 16 / int(sizeof(T));             // values per 16-byte load
         const int n_c = (dv + KC - 1) / KC;                  // channel passes of a thread (dv <= 2 KC)
         float o0[GB], o1[GB];
 #pragma unroll
         for (int gq = 0; gq < GB; gq++) o0[gq] = o1[gq] = 0.0f;
-        for (int js = j0; js <= j1; js += VT) {
-            const int nj = min(VT, j1 - js + 1);
-            const int per_row = dv / PER;
-            __syncthreads();                                 // the last sub-tile has been read
-            for (int i = tid; i < nj * per_row; i += KC) {
-                const int jj = i / per_row, e = (i - jj * per_row) * PER;
-                *reinterpret_cast<uint4*>(vt + jj * dv + e) = *reinterpret_cast<const uint4*>(v_cache + rowoff[js + jj] * dv + e);
+        const T* vt0 = vt;
+        if (vec_v == 2) asm volatile("cp.async.wait_all;" ::: "memory");
+        const int step_v = vec_v == 2 ? KC : VT;
+        for (int js = j0; js <= j1; js += step_v) {
+            const int nj = min(step_v, j1 - js + 1);
+            __syncthreads();                                 // the last sub-tile has been read (2: everybody's copies are there)
+            if (vec_v == 1) {
+                const int per_row = dv / PER;
+                for (int i = tid; i < nj * per_row; i += KC) {
+                    const int jj = i / per_row, e = (i - jj * per_row) * PER;
+                    *reinterpret_cast<uint4*>(vt + jj * dv + e) = *reinterpret_cast<const uint4*>(v_cache + rowoff[js + jj] * dv + e);
+                }
+                __syncthreads();
             }
-            __syncthreads();
+            const T* vt = vec_v == 2 ? vt0 + js * dv : vt0;
             if (n_c > 1) {
                 for (int jj = 0; jj < nj; jj++) {
                     const float va = tid < dv ? ib::to_f32(vt[jj * dv + tid]) : 0.0f;
@@ -1143,6 +1162,85 @@ state_scan_kernel(const float* __restrict__ rows, int64_t ld, int q_col, int k_c
     }
 }
 
+// MODE 5 for steps of one token per request: a CTA per (segment, head, 128 columns), a thread for four neighbouring columns and
+// R of the state's rows, whose 16-byte pieces are all on their way at once. Every element, and every read-out's order of
+// additions (R rows in four chains, then the eight groups of rows pairwise), is the scan's: the same bits. The last warp has
+// the column of ones.
+template <int R>
+__global__ void __launch_bounds__(288)
+state_step_kernel(const float* __restrict__ rows, int64_t ld, int q_col, int k_col, int v_col, const float* __restrict__ aux, int64_t lda,
+                  int aux_col, float* __restrict__ state, const int* __restrict__ seg_start, const int* __restrict__ seg_slot,
+                  float* __restrict__ raw_out, int n_heads, int heads_per_qk, int d, int dv, int write_state, const float* __restrict__ skip_w,
+                  float* __restrict__ ones_state, float* __restrict__ ones_out) {
+    __shared__ __align__(16) float qs[LK * R], ks[LK * R];
+    __shared__ __align__(16) float part[LK][132];
+    const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, hq = h / heads_per_qk;
+    ib::pdl_wait();
+    const int64_t t = seg_start[s], slot_head = int64_t(seg_slot[s]) * n_heads + h;
+    const float* row = rows + t * ld;
+    const int lk = tid >> 5, quad = tid & 31, k0 = lk * R;
+    const int col = blockIdx.z * 128 + quad * 4;
+    const bool ones = lk == LK;
+    const bool live = !ones && col < dv;
+    float* S_g = state + slot_head * int64_t(d) * dv + col;
+    float4 S[R];
+    if (live) {
+#pragma unroll
+        for (int i = 0; i < R; i++) S[i] = k0 + i < d ? *reinterpret_cast<const float4*>(S_g + int64_t(k0 + i) * dv) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    const float g = aux[t * lda + aux_col + h], beta = aux[t * lda + aux_col + n_heads + h];
+    for (int i = tid; i < LK * R; i += blockDim.x) {
+        qs[i] = i < d ? row[q_col + hq * d + i] : 0.0f;
+        ks[i] = i < d ? row[k_col + hq * d + i] : 0.0f;
+    }
+    const float4 x = live ? *reinterpret_cast<const float4*>(row + v_col + h * dv + col) : make_float4(1.f, 1.f, 1.f, 1.f);
+    const float4 v = make_float4(beta * x.x, beta * x.y, beta * x.z, beta * x.w);
+    __syncthreads();
+    if (live) {
+        float4 p[4];
+#pragma unroll
+        for (int c = 0; c < 4; c++) p[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < R; i++) {
+            const float k = ks[k0 + i], q = qs[k0 + i];
+            S[i].x = fmaf(g, S[i].x, k * v.x); S[i].y = fmaf(g, S[i].y, k * v.y);
+            S[i].z = fmaf(g, S[i].z, k * v.z); S[i].w = fmaf(g, S[i].w, k * v.w);
+            float4& pc = p[i & 3];
+            pc.x = fmaf(S[i].x, q, pc.x); pc.y = fmaf(S[i].y, q, pc.y); pc.z = fmaf(S[i].z, q, pc.z); pc.w = fmaf(S[i].w, q, pc.w);
+        }
+        if (write_state) {
+#pragma unroll
+            for (int i = 0; i < R; i++)
+                if (k0 + i < d) *reinterpret_cast<float4*>(S_g + int64_t(k0 + i) * dv) = S[i];
+        }
+        *reinterpret_cast<float4*>(&part[lk][quad * 4]) = make_float4((p[0].x + p[1].x) + (p[2].x + p[3].x), (p[0].y + p[1].y) + (p[2].y + p[3].y),
+                                                                      (p[0].z + p[1].z) + (p[2].z + p[3].z), (p[0].w + p[1].w) + (p[2].w + p[3].w));
+    } else if (ones && ones_state && blockIdx.z == 0) {
+        const int j0 = (quad & (LK - 1)) * R;                // eight lanes with R rows each (the other lanes repeat them)
+        float* n_g = ones_state + slot_head * d;
+        float p[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+        for (int i = 0; i < R; i++) {
+            const int r = j0 + i;
+            float n = r < d ? n_g[r] : 0.0f;
+            n = fmaf(g, n, ks[r] * beta);
+            p[i & 3] = fmaf(n, qs[r], p[i & 3]);
+            if (write_state && quad < LK && r < d) n_g[r] = n;
+        }
+        float sum = (p[0] + p[1]) + (p[2] + p[3]);
+        sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+        sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+        sum += __shfl_xor_sync(0xffffffffu, sum, 4);
+        if (quad == 0) ones_out[t * n_heads + h] = sum;
+    }
+    __syncthreads();
+    const int c = blockIdx.z * 128 + tid;
+    if (tid < 128 && c < dv) {
+        const float o = ((part[0][tid] + part[1][tid]) + (part[2][tid] + part[3][tid])) + ((part[4][tid] + part[5][tid]) + (part[6][tid] + part[7][tid]));
+        const float skip = skip_w ? skip_w[h] : 0.0f;
+        raw_out[(t * n_heads + h) * int64_t(dv) + c] = fmaf(skip, row[v_col + h * dv + c], o);
+    }
+}
+
 // One warp per (token, head): out = o / sqrt(mean(o^2) + eps) * w [* silu(gate)], lanes striding over the columns; the
 // gate's logits are columns gate_col + h dv + j of rows `gate` (leading dimension ldg).
 template <typename TG, typename TOut>
@@ -1258,10 +1356,10 @@ IB_EXPORT int ib_route_rows(const void* x, const void* w, int64_t n_tokens, int 
         top > keep * (n_experts / n_groups) || (group_best != 1 && group_best != 2))
         return ib::fail(IB_ERR_ARG, "ib_route_rows: %d experts in %d groups, %d kept, %d chosen", n_experts, n_groups, keep, top);
     if (width <= 0 || width % 8 || ((uintptr_t(x) | uintptr_t(w)) & 15)) return ib::fail(IB_ERR_ARG, "ib_route_rows: rows of %d are not whole 16-byte pieces", width);
-    const size_t smem = size_t(4) * (n_experts + n_groups) * sizeof(float);
     const int eb = n_experts <= 8 ? 8 : (n_experts <= 16 ? 16 : (n_experts <= 32 ? 32 : 64));
+    const size_t smem = (size_t(n_experts) + n_groups + 4 * eb) * sizeof(float);
 #define IB_RR(TT, EE)                                                                                                                \
-    IB_LAUNCH((route_rows_kernel<TT, EE>), blocks_for(n_tokens, 4), 128, smem, (const TT*)x, (const TT*)w, n_tokens, width, n_experts, \
+    IB_LAUNCH((route_rows_kernel<TT, EE>), unsigned(n_tokens), 128, smem, (const TT*)x, (const TT*)w, width, n_experts, \
               top, n_groups, keep, sum_eps, sigmoid, group_best, renormalise, mult, weights, chosen)
 #define IB_RR_BY(TT)                                                                                                                 \
     do {                                                                                                                             \
@@ -1319,8 +1417,10 @@ IB_EXPORT int ib_attention_split(const void* q, const void* k_cache, const void*
     const size_t item = dtype == IB_F32 ? 4 : 2;
     size_t smem = size_t(group * ((d + 3) & ~3) + group * KC + 2 * GMAX) * sizeof(float) + KC * sizeof(int64_t);
     // values through shared memory where a row is whole 16-byte pieces and at most two channels fall to a thread
-    const int vec_v = (dv * item) % 16 == 0 && dv <= 2 * KC && !(uintptr_t(v_cache) & 15) && smem + size_t(VT) * dv * item <= 48 * 1024;
-    if (vec_v) smem += size_t(VT) * dv * item;
+    // (2: a whole chunk's rows at once, where they fit)
+    int vec_v = (dv * item) % 16 == 0 && dv <= 2 * KC && !(uintptr_t(v_cache) & 15) && smem + size_t(VT) * dv * item <= 48 * 1024;
+    if (vec_v && smem + size_t(KC) * dv * item <= 48 * 1024) vec_v = 2;
+    if (vec_v) smem += size_t(vec_v == 2 ? KC : VT) * dv * item;
     if (smem > 48 * 1024) return ib::fail(IB_ERR_ARG, "ib_attention_split: %d heads of %d do not fit", group, d);
     const dim3 grid{unsigned(n_tokens), unsigned(n_kv), unsigned(n_chunks)};
     const int64_t rows = n_tokens * n_heads;
@@ -1410,18 +1510,29 @@ static int launch_scan(dim3 grid, int threads, size_t smem, cudaStream_t stream,
 // before the write and `bonus` [heads, d] on the current token; mode 4: delta rule with decays as mode 0 and beta, k.q at
 // scal_col of the aux rows; mode 5: a decay and a write strength per head and token (aux: at aux_col + h and aux_col + H + h),
 // skip [heads] in `bonus` (null: none), with ones_state and ones_out a column of ones beside the values.
+// `single`: every segment is one token (mode 5 then has a kernel of its own for sizes of whole 16-byte pieces, same bits).
 // `spread` (prompt portions): a head's columns go to more, smaller CTAs until there is about one per SM (sm_count).
 IB_EXPORT int ib_state_scan(int mode, const float* rows, int64_t ld, int q_col, int k_col, int v_col, const float* aux,
                             int64_t lda, int aux_col, float* state, const int* seg_start, const int* seg_slot,
                             float* raw_out, int n_segments, int n_heads, int heads_per_qk, int d, int dv, int write_state,
                             int spread, int sm_count, cudaStream_t stream, const float* bonus, int act, int scal_col,
-                            float* ones_state, float* ones_out) {
+                            float* ones_state, float* ones_out, int single) {
     if (n_segments <= 0) return IB_OK;
     if (n_heads <= 0 || n_heads > 65535 || heads_per_qk <= 0 || n_heads % heads_per_qk || d <= 0 || dv <= 0 || d > LK * 32)
         return ib::fail(IB_ERR_ARG, "ib_state_scan: %d heads with a state of %d x %d do not fit", n_heads, d, dv);
     if (mode < 0 || mode > 5) return ib::fail(IB_ERR_ARG, "ib_state_scan: unknown mode %d", mode);
     if (mode == 3 && !bonus) return ib::fail(IB_ERR_ARG, "ib_state_scan: mode 3 needs the bonus");
     if (ones_state && (mode != 5 || !ones_out)) return ib::fail(IB_ERR_ARG, "ib_state_scan: a column of ones goes with mode 5 and a result of its own");
+    if (mode == 5 && single && !act && dv % 4 == 0 && ld % 4 == 0 && v_col % 4 == 0 && !((uintptr_t(rows) | uintptr_t(state)) & 15)) {
+        const int r1 = d <= 32 ? 4 : (d <= 64 ? 8 : (d <= 128 ? 16 : 32));
+        const dim3 grid1{unsigned(n_segments), unsigned(n_heads), unsigned((dv + 127) / 128)};
+#define IB_STEP(RR)                                                                                                                   \
+        IB_LAUNCH(state_step_kernel<RR>, grid1, 288, 0, rows, ld, q_col, k_col, v_col, aux, lda, aux_col, state, seg_start, seg_slot, \
+                  raw_out, n_heads, heads_per_qk, d, dv, write_state, bonus, ones_state, ones_out)
+        if (r1 == 4) IB_STEP(4); else if (r1 == 8) IB_STEP(8); else if (r1 == 16) IB_STEP(16); else IB_STEP(32);
+#undef IB_STEP
+        return ib::check_launch("ib_state_scan");
+    }
     const bool decay_rows = mode == 0 || mode == 3 || mode == 4;
     const int columns = dv + (ones_state ? 1 : 0);
     const int r = d <= 32 ? 4 : (d <= 64 ? 8 : (d <= 128 ? 16 : 32));

@@ -864,11 +864,11 @@ def state_scan(mode: int, rows: torch.Tensor, q_col: int, k_col: int, v_col: int
     spread = int(max_len) >= SCAN_SPREAD_FROM
     sm_count = torch.cuda.get_device_properties(rows.device).multi_processor_count if spread else 0
     f = _fn("mix", "ib_state_scan", [c_int, c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_int64, c_int, c_void_p, c_void_p,
-                                     c_void_p, c_void_p] + [c_int] * 8 + [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p])
+                                     c_void_p, c_void_p] + [c_int] * 8 + [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int])
     _call(f, int(mode), rows.data_ptr(), ld, int(q_col), int(k_col), int(v_col), aux.data_ptr(), lda, int(aux_col),
           state.data_ptr(), seg_start.data_ptr(), seg_slot.data_ptr(), out.data_ptr(), S, n_heads, int(heads_per_qk), dim, v_dim,
           int(write_state), int(spread), sm_count, _stream(), _ptr(bonus) if mode in (SCAN_BONUS, SCAN_STEP) else None, int(bool(silu)),
-          int(scalar_col), _ptr(ones_state), _ptr(ones_out))
+          int(scalar_col), _ptr(ones_state), _ptr(ones_out), int(max_len == 1))
     return out if ones_state is None else (out, ones_out)
 
 

@@ -272,8 +272,10 @@ def test_scan_with_a_decay_and_a_strength_per_token_over_steps(sizes, ones):
     assert bool(torch.isnan(state[1]).all()) and bool(torch.isnan(n_state).all(dim=-1)[1].all())
 
 
-def test_step_scan_cuttings_are_bit_equal():
-    H, G, d, dv, n = 2, 1, 40, 24, 45
+@pytest.mark.parametrize("d,dv", [(40, 24), (128, 128), (64, 132), (16, 260), (200, 8), (33, 9)])
+def test_step_scan_cuttings_are_bit_equal(d, dv):
+    """Whole, in portions, and one token at a time (which has a kernel of its own where a row is whole 16-byte pieces)."""
+    H, G, n = 2, 1, 45
     seqs = _step_case(H, G, d, dv, 9, (n, 3))
     outs = []
     for cuts in ([45], [1] * 45, [2] * 22 + [1], [7, 30, 8]):
