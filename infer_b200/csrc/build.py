@@ -36,6 +36,7 @@ MODULES: Dict[str, str] = {
     "stream": "stream_ops.cu",   # several residual streams, norms over groups of channels, sinusoidal positions
     "memory": "memory_ops.cu",   # scaled sums with the next norm, state space layers' filters and steps, matrix memories' gates
     "chunk": "chunk_scan.cu",    # the recurrences of the two lines above over prompt portions, in chunks on the tensor cores
+    "experts": "expert_ops.cu",  # rows gathered by expert, around the grouped products of a routed feed-forward
     "talk": "talk_ops.cu",       # attention whose heads exchange their scores before the softmax
     "talk_pf": "talk_prefill.cu",       # the same attention for prompt portions on the tensor cores
     "latent_pf": "latent_prefill.cu",   # the same attention for prompt portions: per-head keys and values, tensor cores

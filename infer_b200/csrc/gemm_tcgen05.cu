@@ -213,6 +213,10 @@ struct GemmParams {
     int recv_in_ring;                    // 1: the slices' columns are received in the operand ring itself, once every slice
                                          //    of the cluster is done with its ring (one more cluster barrier; for tiles whose
                                          //    float columns would not fit behind the ring)
+    // grouped products (GROUPED persistent kernel): the row tiles in use and the expert of each, [0] count, [1 + i]; which B rows
+    // and which first k a tile's expert has: row (tn / g_tph) * g_half + expert * g_rows + (tn % g_tph) * width, k = expert * g_k
+    const int* tiles;
+    int g_tiles_n, g_tph, g_half, g_rows, g_k;
 };
 
 template <int BN> struct Cfg {
@@ -758,7 +762,7 @@ __device__ __forceinline__ void drain_row(const GemmParams& p, uint32_t taddr, i
     }
 }
 
-template <int PBN, bool WIDE, typename TOut>
+template <int PBN, bool WIDE, typename TOut, bool GROUPED = false>
 __global__ void __launch_bounds__(NUM_THREADS)
 gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_constant__ CUtensorMap tm_b, const GemmParams p) {
     extern __shared__ uint8_t smem_raw[];
@@ -774,8 +778,16 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid
     volatile uint32_t* slots = reinterpret_cast<volatile uint32_t*>(base_ptr + S * P_STAGE_BYTES + (2 * S + 4) * 8);
     // slots[0] = TMEM base address, slots[1] = abort flag
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int tiles_m = int((p.rows_a + TM - 1) / TM), tiles_n = int((p.rows_b + TN - 1) / TN);
-    const int n_tiles = tiles_m * tiles_n;
+    int tiles_m = int((p.rows_a + TM - 1) / TM);
+    const int tiles_n = GROUPED ? p.g_tiles_n : int((p.rows_b + TN - 1) / TN);
+    int n_tiles = tiles_m * tiles_n;
+    // (a predecessor writes the table: every role asks once it may read)
+    auto tiles_in_use = [&]() {
+        if constexpr (GROUPED) {
+            tiles_m = min(tiles_m, *reinterpret_cast<const volatile int*>(p.tiles));
+            n_tiles = tiles_m * tiles_n;
+        }
+    };
     const int n_kb = p.kb_total;
     auto full_bar = [&](int s) { return bars + 8u * s; };
     auto empty_bar = [&](int s) { return bars + 8u * (S + s); };
@@ -804,10 +816,17 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid
         if (p.early_release && lane != 0) ib::pdl_launch_dependents();
         if (lane == 0) {
             ib::pdl_wait();
+            tiles_in_use();
             int it = 0, issued = 0;
             const uint64_t once = policy_evict_first();
             for (int tile = blockIdx.x; tile < n_tiles && !slots[1]; tile += gridDim.x) {
                 const int tm = tile % tiles_m, tn = tile / tiles_m;    // neighbouring CTAs share the weight tile
+                int b_row = tn * TN, b_k = 0;
+                if constexpr (GROUPED) {
+                    const int e = p.tiles[1 + tm];
+                    b_row = (tn / p.g_tph) * p.g_half + e * p.g_rows + (tn % p.g_tph) * TN;
+                    b_k = e * p.g_k;
+                }
                 for (int kb = 0; kb < n_kb; kb++, it++) {
                     const int s = it % S;
                     if (it >= S && !mbar_wait(empty_bar(s), ((it / S) - 1) & 1)) {
@@ -817,8 +836,8 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid
                     const uint32_t a_dst = base + s * P_STAGE_BYTES, b_dst = a_dst + A_BYTES;
                     mbar_expect_tx(full_bar(s), A_BYTES + B_BYTES);
                     tma_load_2d(a_dst, &tm_a, full_bar(s), kb * BK, tm * TM);
-                    if (p.weights_once) tma_load_2d_once(b_dst, &tm_b, full_bar(s), kb * BK, tn * TN, once);
-                    else tma_load_2d(b_dst, &tm_b, full_bar(s), kb * BK, tn * TN);
+                    if (p.weights_once) tma_load_2d_once(b_dst, &tm_b, full_bar(s), b_k + kb * BK, b_row, once);
+                    else tma_load_2d(b_dst, &tm_b, full_bar(s), b_k + kb * BK, b_row);
                     issued = it + 1;
                 }
             }
@@ -832,6 +851,8 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid
         if (lane == 0) {
             constexpr uint32_t idesc = make_idesc(TN);
             int it = 0, lt = 0;
+            if constexpr (GROUPED) ib::pdl_wait();
+            tiles_in_use();
             for (int tile = blockIdx.x; tile < n_tiles && !slots[1]; tile += gridDim.x, lt++) {
                 const int b = lt & 1;
                 if (lt >= 2 && !mbar_wait(acc_empty_bar(b), ((lt >> 1) - 1) & 1)) {      // the epilogue has drained it
@@ -868,6 +889,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid
         // ---------------------------------------------------------------- epilogue (warps 2..5)
         const int quad = warp & 3;
         ib::pdl_wait();
+        tiles_in_use();
         int lt = 0;
         ResidualAhead ra;
         for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x, lt++) {
@@ -1079,7 +1101,7 @@ IB_EXPORT int ib_gemm_tc(const void* x, const void* w, const float* bias, const 
     if (!status) return ib::fail(IB_ERR_ARG, "gemm_tc: a status word is required");
     if (epi != 0 && epi != 2) return ib::fail(IB_ERR_ARG, "gemm_tc: unknown epilogue %d", epi);
     if (epi == 2 && (N % 16 || bias || residual)) return ib::fail(IB_ERR_ARG, "gemm_tc: the SwiGLU epilogue needs N %% 16 == 0 and no bias or residual");
-    GemmParams p;
+    GemmParams p = {};
     p.epi = epi;
     p.swap = swap ? 1 : 0;
     p.M = M; p.N = N; p.K = K;
@@ -1145,6 +1167,74 @@ IB_EXPORT int ib_gemm_tc(const void* x, const void* w, const float* bias, const 
         case 64: return f32 ? launch<64, float>(ma, mb, p, grid, stream) : launch<64, bf16>(ma, mb, p, grid, stream);
         default: return f32 ? launch<128, float>(ma, mb, p, grid, stream) : launch<128, bf16>(ma, mb, p, grid, stream);
     }
+}
+
+// A product whose rows are grouped by expert (expert_ops.cu): x [max_tiles * 128, K] bfloat16, a whole number of 128-row tiles an
+// expert, tiles [0] = the tiles in use and tiles[1 + i] the expert of tile i, in device memory. w bfloat16 is one matrix for all
+// experts. side 0 (an expert's rows of a stack of `halves` matrices [experts * n_expert, K]): out [rows, halves * padded],
+// padded = n_expert rounded up to the kernel's width (returned in *padded; the columns beyond n_expert are not meaningful);
+// side 1 (an expert's columns, [N, experts * K]): out [rows, N]. With x null only *padded is computed.
+IB_EXPORT int ib_gemm_tc_grouped(const void* x, const void* w, void* out, int64_t max_tiles, int64_t likely_tiles, int64_t n_expert, int64_t K,
+                                 int n_experts, int halves, int side, const int* tiles, int out_dtype, int sm_count, int* status,
+                                 int64_t* padded, cudaStream_t stream) {
+    if (max_tiles <= 0 || n_expert <= 0 || K <= 0 || n_experts <= 0 || halves < 1 || (side != 0 && side != 1))
+        return ib::fail(IB_ERR_ARG, "gemm_tc_grouped: sizes must be positive");
+    if (K % 8) return ib::fail(IB_ERR_ARG, "gemm_tc_grouped: K = %lld is not a multiple of 8", (long long)K);
+    const int64_t sms = sm_count > 0 ? sm_count : 148;
+    // as for the other persistent products: rounds over the SMs times (width + 224)
+    int width = 256;
+    int64_t best = -1;
+    for (int wd : {256, 192}) {
+        const int64_t t = (likely_tiles > 0 ? likely_tiles : max_tiles) * halves * ((n_expert + wd - 1) / wd);
+        const int64_t cost = ((t + sms - 1) / sms) * (wd + 224);
+        if (best < 0 || cost < best) { best = cost; width = wd; }
+    }
+    const int64_t tph = (n_expert + width - 1) / width;
+    if (padded) *padded = side == 0 ? tph * width : n_expert;
+    if (!x) return IB_OK;
+    if (!w || !out || !tiles || !status) return ib::fail(IB_ERR_ARG, "gemm_tc_grouped: operands, result, table and status are needed");
+    if (((uintptr_t(x) | uintptr_t(w) | uintptr_t(out)) & 15)) return ib::fail(IB_ERR_ARG, "gemm_tc_grouped: operand bases must be 16-byte aligned");
+    if (out_dtype != IB_F32 && out_dtype != IB_BF16) return ib::fail(IB_ERR_ARG, "gemm_tc_grouped: unknown output dtype %d", out_dtype);
+    const int64_t rows = max_tiles * 128, b_rows = side == 0 ? int64_t(halves) * n_experts * n_expert : n_expert;
+    const int64_t b_cols = side == 0 ? K : int64_t(n_experts) * K;
+    if (rows >= (1LL << 31) || b_rows >= (1LL << 31) || b_cols >= (1LL << 31)) return ib::fail(IB_ERR_ARG, "gemm_tc_grouped: a size exceeds 2^31");
+    GemmParams p = {};
+    p.rows_a = rows; p.rows_b = b_rows; p.K = K;
+    p.kb_total = int((K + BK - 1) / BK);
+    p.kb_per_split = p.kb_total; p.splits = 1; p.stages = PSTAGES;
+    p.M = rows; p.N = side == 0 ? halves * tph * width : n_expert;
+    p.out = out; p.status = status; p.early_release = 1;
+    p.tiles = tiles;
+    p.g_tph = int(tph);
+    p.g_tiles_n = int(halves * tph);
+    p.g_half = side == 0 ? int(n_experts * n_expert) : 0;
+    p.g_rows = side == 0 ? int(n_expert) : 0;
+    p.g_k = side == 0 ? 0 : int(K);
+    if (side == 1 && halves != 1) return ib::fail(IB_ERR_ARG, "gemm_tc_grouped: an expert's columns are one matrix");
+    CUtensorMap ma, mb;
+    int rc = get_map(x, rows, K, 128, &ma);
+    if (rc) return rc;
+    rc = get_map(w, b_rows, b_cols, width, &mb);
+    if (rc) return rc;
+#define IB_GROUPED(WW, TT)                                                                                                           \
+    do {                                                                                                                             \
+        static bool configured = false;                                                                                              \
+        if (!configured) {                                                                                                           \
+            cudaError_t e = cudaFuncSetAttribute(gemm_tc_persistent_kernel<WW, true, TT, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, P_SMEM_BYTES); \
+            if (e != cudaSuccess) return ib::fail(IB_ERR_CUDA, "gemm_tc_grouped: cannot set shared memory size: %s", cudaGetErrorString(e)); \
+            configured = true;                                                                                                       \
+        }                                                                                                                            \
+        const int64_t most = max_tiles * p.g_tiles_n;                                                                                \
+        return ib::launch("gemm_tc_grouped", gemm_tc_persistent_kernel<WW, true, TT, true>, dim3(unsigned(most < sms ? most : sms)), \
+                          dim3(NUM_THREADS), size_t(P_SMEM_BYTES), stream, 1u, ma, mb, p);                                           \
+    } while (0)
+    if (width == 256) {
+        if (out_dtype == IB_F32) IB_GROUPED(256, float);
+        IB_GROUPED(256, bf16);
+    }
+    if (out_dtype == IB_F32) IB_GROUPED(192, float);
+    IB_GROUPED(192, bf16);
+#undef IB_GROUPED
 }
 
 // ================================================================================================

@@ -204,6 +204,75 @@ def linear(x, weight, bias, residual, out_dtype, out, swiglu=False):
     return gemm_tc(x, weight, bias, residual, out_dtype, out, swiglu=swiglu)
 
 
+GROUPED_FROM = 256            # tokens from which a routed feed-forward's rows are worth grouping by expert
+
+
+def grouped_experts_worth(n_tokens: int, top: int, n_experts: int) -> bool:
+    """True where the chosen experts' rows, each expert's padded to whole tiles, are well below tokens x experts."""
+    return n_tokens >= GROUPED_FROM and 5 * (n_tokens * top + 64 * n_experts) <= 3 * n_tokens * n_experts
+
+
+class RowGroups:
+    """The rows of a step that each expert was chosen for, side by side (``ops``-level view of the grouping kernels): ``place`` int32
+    [T, top], ``scale`` float32 [rows, 1] (the token's weight for the row's expert), the table of tiles."""
+
+    def __init__(self, weights: torch.Tensor, chosen: torch.Tensor):
+        _check(weights, "weights", torch.float32)
+        _check(chosen, "chosen", torch.int32)
+        self.T, self.top = chosen.shape
+        self.E = weights.shape[1]
+        tile = int(_fn("experts", "ib_group_tile_rows", [])())
+        pairs = self.T * self.top
+        self.max_tiles = pairs // tile + min(self.E, pairs)
+        self.likely_tiles = min(self.max_tiles, -(-pairs // tile) + self.E // 2)
+        self.rows = self.max_tiles * tile
+        dev = weights.device
+        self.place = torch.empty(pairs, dtype=torch.int32, device=dev)
+        self.row_of = torch.empty(self.rows, dtype=torch.int32, device=dev)
+        self.scale = torch.empty((self.rows, 1), dtype=torch.float32, device=dev)
+        self.tiles = torch.empty(1 + self.max_tiles, dtype=torch.int32, device=dev)
+        f = _fn("experts", "ib_group_rows", [c_void_p, c_void_p, c_int64, c_int, c_int] + [c_void_p] * 5)
+        _call(f, chosen.data_ptr(), weights.data_ptr(), self.T, self.top, self.E, self.place.data_ptr(), self.row_of.data_ptr(),
+              self.scale.data_ptr(), self.tiles.data_ptr(), _stream())
+
+    def gather(self, x: torch.Tensor) -> torch.Tensor:
+        """[rows, W]: x's row of each grouped row (zeros in the padding; rows of tiles that are not in use are left as they are)."""
+        _check(x, "x", torch.bfloat16)
+        out = torch.empty((self.rows, x.shape[1]), dtype=x.dtype, device=x.device)
+        f = _fn("experts", "ib_gather_rows", [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int64, c_void_p])
+        _call(f, x.data_ptr(), self.row_of.data_ptr(), self.tiles.data_ptr(), out.data_ptr(), self.rows, x.shape[1] * 2, _stream())
+        return out
+
+    def product(self, x: torch.Tensor, w: torch.Tensor, n_expert: int, halves: int, side: int, out_dtype: torch.dtype):
+        """x [rows, K] times its expert's part of w. side 0: w [halves * E * n_expert, K] (an expert's rows of each half), result
+        [rows, halves * padded], returned with padded; side 1: w [n_expert, E * K] (an expert's columns), result [rows, n_expert]."""
+        _check(x, "x", torch.bfloat16)
+        _check(w, "w", torch.bfloat16)
+        K = x.shape[1]
+        want = (halves * self.E * n_expert, K) if side == 0 else (n_expert, self.E * K)
+        if x.shape[0] != self.rows or tuple(w.shape) != want:
+            raise KernelError(f"grouped product: x {tuple(x.shape)}, w {tuple(w.shape)}, expected {self.rows} rows and {want}")
+        st = device_state(x.device)
+        f = _fn("gemm", "ib_gemm_tc_grouped", [c_void_p] * 3 + [c_int64] * 4 + [c_int] * 3 + [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p])
+        padded = ctypes.c_int64(0)
+        args = [self.max_tiles, self.likely_tiles, n_expert, K, self.E, halves, side, self.tiles.data_ptr(), dtype_code(out_dtype), st.sm_count,
+                st.status.data_ptr(), ctypes.addressof(padded), _stream()]
+        if f(None, w.data_ptr(), None, *args):
+            raise KernelError("grouped product: " + f._lib.ib_last_error().decode())
+        out = torch.empty((self.rows, halves * padded.value), dtype=out_dtype, device=x.device)
+        _call(f, x.data_ptr(), w.data_ptr(), out.data_ptr(), *args)
+        return out, padded.value
+
+    def combine(self, y: torch.Tensor, residual: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """float32 [T, W]: (residual +) the sum of each token's rows, over ``residual`` where given."""
+        _check(y, "y", torch.float32)
+        W = y.shape[1]
+        out = residual if residual is not None else torch.empty((self.T, W), dtype=torch.float32, device=y.device)
+        f = _fn("experts", "ib_combine_rows", [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int64, c_int64, c_void_p])
+        _call(f, y.data_ptr(), self.place.data_ptr(), self.top, _ptr(residual), out.data_ptr(), self.T, W, _stream())
+        return out
+
+
 def attention_supported(n_heads: int, n_kv: int, head_dim: int, page_size: int) -> bool:
     return head_dim % 16 == 0 and 16 <= head_dim <= 128 and page_size == 16 and n_heads // n_kv <= 16
 

@@ -13,7 +13,8 @@ kernel multiplies an expert's hidden values by the token's weight for that exper
 token does not use; one product with the experts' down matrices side by side then sums the chosen experts. Every
 expert's matrices are read once per step whatever the routing, which is what a batch of decoding requests or a prompt
 portion does anyway; the multiply-adds of experts a token does not use are spent for nothing (experts / top times the
-needed ones).
+needed ones). For prompt portions of some hundred tokens and few chosen experts the rows are gathered by expert instead, and
+the products run over each expert's rows only (``fast_ops.RowGroups``).
 
 Tensors: ``router`` [experts, hidden]; per expert i ``e<i>.gate``, ``e<i>.up`` [ff, hidden], ``e<i>.down`` [hidden, ff];
 ``shared.gate`` / ``shared.up`` / ``shared.down`` likewise. No biases.
@@ -115,6 +116,8 @@ class RoutedExperts(FeedForward):
 
     def forward(self, x, residual, side_stream=None):
         """With ``side_stream`` the router runs there, beside the experts' first product (forked and joined here)."""
+        if self._groups_rows(x):
+            return self._forward_grouped(x, residual)
         if side_stream is None:
             return self._experts(self._weights(x), self.gate_up(x), residual)
         main = torch.cuda.current_stream(x.device)
@@ -128,15 +131,39 @@ class RoutedExperts(FeedForward):
         main.wait_event(done)
         return self._experts(weights, rows, residual)
 
+    def _groups_rows(self, x) -> bool:
+        """Prompt portions, where a token's chosen experts are few: the rows are gathered by expert, and the tokens go
+        through the chosen experts only (tensor-core products of rows of 16-byte pieces)."""
+        if self.rt.dtype != torch.bfloat16 or not self.rt.fast("linear") or self.shared_ff or self.expert_kind == "relu_squared" \
+                or self.router_kind == "sigmoid" or self.hidden % 8 or self.ff % 8:
+            return False
+        from .. import fast_ops
+        return fast_ops.grouped_experts_worth(x.shape[0], self.top, self.n_experts)
+
+    def _forward_grouped(self, x, residual):
+        from .. import fast_ops
+        got = self._route(x, True)
+        groups = fast_ops.RowGroups(*got)
+        rows, up = groups.product(groups.gather(x), self.gate_up.weight, self.ff, 2, 0, self.rt.dtype)
+        act = ops.glu_act(rows, 0, up, self.ff, "swish" if self.expert_kind == "swish_glu" else "clipped_swish", self.limit, self.limit,
+                          self.slope, groups.scale, self.ff, 1)
+        y, _ = groups.product(act, self.down.weight, self.hidden, 1, 1, torch.float32)
+        return groups.combine(y, residual)
+
     def _weights(self, x):
         if self.router_kind == "sigmoid":
             return ops.route_sigmoid(self.router(x, out_dtype=torch.float32), self.correction, self.top, self.out_scale)[0]
+        return self._route(x)[0]
+
+    def _route(self, x, want_chosen=False):
+        """(weights [T, experts], chosen [T, top] if asked for)."""
         how = dict(sigmoid=True, group_best=2, renormalise=False, mult=self.out_scale) if self.router_kind == "sigmoid_groups" \
             else dict(sum_eps=self.sum_eps)
+        how["want_chosen"] = want_chosen
         got = ops.route_rows(x, self.router.weight, self.top, self.groups, self.keep, **how)      # the product in the same kernel
         if got is None:
             got = ops.route(self.router(x, out_dtype=torch.float32), self.top, self.groups, self.keep, **how)
-        return got[0]
+        return got
 
     def _experts(self, weights, rows, residual):
         if self.expert_kind == "relu_squared":

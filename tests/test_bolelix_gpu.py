@@ -184,6 +184,20 @@ def test_a_batch_of_unequal_requests_equals_each_alone():
             assert np.array_equal(alone[r][p], together[r][p])
 
 
+def test_long_prompts_run_chunked_scans_and_grouped_experts():
+    """A prompt of 300 tokens, and the same tokens in portions: the scans take 64 tokens at a time, routed layers with few chosen
+    experts gather their rows; results as for every other way of running them."""
+    from infer_b200 import ops
+    cfg = BC.CASES["c"]
+    ids = BC.random_ids(cfg, 420, 91)
+    before = dict(ops.LAUNCH_KINDS)
+    got = H.run_trace(_engine("c", torch.bfloat16), [{"entries": [("x", ids[:300], list(range(300)))], "end": []},
+                                                     {"entries": [("x", ids[300:], list(range(120)))], "end": ["x"]}])
+    ran = {k: v - before.get(k, 0) for k, v in ops.LAUNCH_KINDS.items() if v != before.get(k, 0)}
+    assert ran.get("ib_chunk_scan", 0) == 8 and ran.get("ib_group_rows", 0) >= 2 and ran["ib_gemm_tc_grouped"] == 2 * ran["ib_group_rows"], ran
+    BC.check(cfg, SEED, torch.bfloat16, got, {"x": ids}, what="long")
+
+
 def test_the_design_runs_on_its_own_kernels():
     from infer_b200 import ops
     eng = _engine("c", torch.bfloat16)

@@ -424,3 +424,40 @@ def test_router_with_its_product(E, top, width, dtype):
     assert torch.allclose(weights.double().cpu()[clear], full[clear], rtol=1e-4, atol=1e-6)
     assert torch.equal(ops.route_rows(x[5:6].to(DEV).contiguous(), w.to(DEV), top)[0][0], weights[5])      # whatever else is in the step
     assert ops.route_rows(torch.zeros(2, 12, device=DEV), torch.zeros(4, 12, device=DEV), 1) is None       # no whole pieces: another path
+
+
+@pytest.mark.parametrize("T,E,top,width,ff", [(300, 8, 2, 128, 72), (256, 16, 4, 64, 16), (513, 8, 1, 136, 200), (700, 5, 2, 1536, 1120), (2048, 8, 2, 256, 264)])
+@pytest.mark.parametrize("with_residual", [False, True])
+def test_products_over_rows_grouped_by_expert(T, E, top, width, ff, with_residual):
+    """Every pair of a token and a chosen expert has one row; experts without a row, with a few, and with several tiles of rows;
+    both grouped products, the gated activation with the token's weight, and the sum over a token's rows."""
+    from infer_b200 import fast_ops
+    g = torch.Generator().manual_seed(T)
+    x = torch.randn(T, width, generator=g).to(torch.bfloat16)
+    z = torch.randn(T, E, generator=g) + torch.linspace(4, -4, E)            # (unequal groups)
+    z[:, E // 2] = -1e9                                                      # one expert that nobody chose
+    chosen, ww, _ = pb.route_top(z.double(), top)
+    weights = torch.zeros(T, E, dtype=F).scatter_(1, chosen, ww)
+    gu = (torch.randn(2 * E * ff, width, generator=g) * width ** -0.5).to(torch.bfloat16)
+    down = (torch.randn(width, E * ff, generator=g) * ff ** -0.5).to(torch.bfloat16)
+    groups = fast_ops.RowGroups(weights.float().to(DEV), chosen.int().to(DEV).contiguous())
+    n_tiles = int(groups.tiles[0])
+    assert n_tiles == sum(-(-int((chosen == e).sum()) // 128) for e in range(E)) <= groups.max_tiles
+    place = groups.place.cpu().view(T, top).long()
+    assert len(set(place.flatten().tolist())) == T * top
+    expert_of = groups.tiles[1:1 + n_tiles].cpu().long()
+    assert torch.equal(expert_of[place // 128], chosen) and torch.equal(groups.row_of.cpu()[place].long(), torch.arange(T)[:, None].expand(T, top))
+    assert torch.allclose(groups.scale.cpu()[place, 0].double(), ww, rtol=1e-6)
+    rows, up = groups.product(groups.gather(x.to(DEV)), gu.to(DEV), ff, 2, 0, torch.bfloat16)
+    act = ops.glu_act(rows, 0, up, ff, "swish", 0.0, 0.0, 1.0, groups.scale, ff, 1)
+    y, _ = groups.product(act, down.to(DEV), width, 1, 1, torch.float32)
+    res = torch.randn(T, width, generator=g) if with_residual else None
+    out = groups.combine(y, res.clone().to(DEV) if res is not None else None).double().cpu()
+    want = res.double() if res is not None else torch.zeros(T, width, dtype=F)
+    for e in range(E):
+        at = (chosen == e).nonzero()
+        t, w = at[:, 0], ww[at[:, 0], at[:, 1]]
+        r = lambda v: v.to(torch.bfloat16).double()
+        gate, upv = (r(x[t].double() @ gu[o + e * ff:o + (e + 1) * ff].double().T) for o in (0, E * ff))
+        want[t] += r(pb.silu(gate) * upv * w[:, None]) @ down[:, e * ff:(e + 1) * ff].double().T
+    assert torch.allclose(out, want, rtol=2e-2, atol=2e-2) and float((out - want).pow(2).mean().sqrt()) < 4e-3
