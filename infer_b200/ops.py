@@ -1621,9 +1621,12 @@ def step_scan(rows: torch.Tensor, q_col: int, k_col: int, v_col: int, aux: torch
     S = step.seg_slot.numel()
     _check(step.seg_start, "seg_start", torch.int32, (S + 1,))
     out = torch.empty((T, n_heads * v_dim), dtype=torch.float32, device=rows.device)
+    n_ws = int(_fn("chunk", "ib_chunk_scan_workspace", [c_int64, c_int, c_int, c_int], restype=c_int64)(T, n_heads, int(heads_per_qk), dim))
+    ws = torch.empty(n_ws, dtype=torch.bfloat16, device=rows.device)
     f = _fn("chunk", "ib_chunk_scan", [c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_int64, c_int, c_int] + [c_void_p] * 7 +
-            [c_int] * 7 + [c_void_p])
+            [c_int] * 7 + [c_void_p, c_int64, c_void_p])
     _call(f, rows.data_ptr(), ld, int(q_col), int(k_col), int(v_col), aux.data_ptr(), aux.shape[1], int(b_col), int(lng_col), state.data_ptr(),
           _ptr(ones_state), step.seg_start.data_ptr(), step.seg_slot.data_ptr(), out.data_ptr(), _ptr(ones_out), _ptr(skip), S, n_heads,
-          int(heads_per_qk), dim, v_dim, int(write_state), torch.cuda.get_device_properties(rows.device).multi_processor_count, _stream())
+          int(heads_per_qk), dim, v_dim, int(write_state), torch.cuda.get_device_properties(rows.device).multi_processor_count,
+          ws.data_ptr(), T, _stream())
     return out if ones_state is None else (out, ones_out)
